@@ -6,6 +6,8 @@
 //   * query head h reads kv head h / (heads / kv_heads);
 //   * score = (q . k) * scale * head_scale[h]  (head_scale optional); with softcap > 0 the score then passes
 //     softcap * tanh(score / softcap);
+//   * optionally a key d positions back loses r1[h] * ln(1 + r2[h] * d) of its score (after the cap), and a sink: one
+//     more number per head that takes its share exp(sink[h]) of the softmax's sum and stands for no key;
 //   * the keys a query at position p sees: max(p - window + 1, floor(p / chunk) * chunk, 0) .. p
 //     (window 0: no window; chunk 0: no chunks) — chunks are counted from position 0 of the sequence;
 //   * optionally, beside a window, one pooled key and value per block of positions that lies wholly before it
@@ -75,7 +77,7 @@ __device__ __forceinline__ float flex_dot<float>(const float* __restrict__ q, co
 template <typename T, int NJ>
 __device__ __forceinline__ void flex_run(const float* __restrict__ q_s, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                                          const PagedKV& kp, const PagedKV& vp, int seq, int kh, int kvh, int lo, int hi, float sc,
-                                         float softcap, int lane, float& m, float& l, float (&acc)[NJ]) {
+                                         float softcap, float r1, float r2, int pos, int lane, float& m, float& l, float (&acc)[NJ]) {
   const int dk = kp.head_dim, dv = vp.head_dim;
   for (int c0 = (lo / 32) * 32; c0 <= hi; c0 += 32) {
     const int s = c0 + lane;
@@ -84,6 +86,7 @@ __device__ __forceinline__ void flex_run(const float* __restrict__ q_s, const T*
     if (valid) {
       score = flex_dot<T>(q_s, k_cache + kv_row_offset(kp, seq, s, kh), dk) * sc;
       if (softcap > 0.f) score = softcap * tanhf(score / softcap);
+      if (r1 != 0.f) score -= r1 * logf(fmaf(r2, (float)(pos - s), 1.0f));
     }
     const float m_new = fmaxf(m, warp_max(score));
     const float p = valid ? expf(score - m_new) : 0.f;
@@ -129,7 +132,8 @@ attention_flex_kernel(const T* __restrict__ q, long ldq, OutT* __restrict__ out,
                       const T* __restrict__ v_cache, const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos,
                       PagedKV kp, PagedKV vp, int n_tokens, int n_heads, int maps, float scale,
                       const float* __restrict__ head_scale, int window, int chunk, PooledKV pooled,
-                      const float* __restrict__ gate, long ldg, int gate_per, float softcap) {
+                      const float* __restrict__ gate, long ldg, int gate_per, float softcap,
+                      const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink) {
   __shared__ float q_s[FLEX_WARPS][FLEX_MAX_DK];
   pdl_launch_dependents();
   pdl_wait();
@@ -163,8 +167,10 @@ attention_flex_kernel(const T* __restrict__ q, long ldq, OutT* __restrict__ out,
 
   const int nb = pooled.k ? pooled_blocks_visible(pos, window, pooled.pool) : 0;
   if (nb > 0)
-    flex_run<T, NJ>(q_s[warp], (const T*)pooled.k, (const T*)pooled.v, pooled.kp, pooled.vp, seq, kh, kvh, 0, nb - 1, sc, softcap, lane, m, l, acc);
-  flex_run<T, NJ>(q_s[warp], k_cache, v_cache, kp, vp, seq, kh, kvh, lo, pos, sc, softcap, lane, m, l, acc);
+    flex_run<T, NJ>(q_s[warp], (const T*)pooled.k, (const T*)pooled.v, pooled.kp, pooled.vp, seq, kh, kvh, 0, nb - 1, sc, softcap, 0.f, 0.f, pos, lane, m, l, acc);
+  flex_run<T, NJ>(q_s[warp], k_cache, v_cache, kp, vp, seq, kh, kvh, lo, pos, sc, softcap, r1 ? r1[h] : 0.f, r2 ? r2[h] : 0.f, pos, lane, m,
+                  l, acc);
+  if (sink) l += expf(sink[h] - m);            // (a sink far above every score: infinity, and the output is 0)
   float inv = 1.0f / l;
   if (gate && gate_per <= 1) inv *= 1.0f / (1.0f + expf(-gate[(size_t)t * ldg + h]));
 #pragma unroll
@@ -256,7 +262,8 @@ template <typename T, typename OutT>
 int launch_attention_flex(const void* q, long ldq, void* out, long ldo, const void* k_cache, const void* v_cache,
                           const int32_t* tok_seq, const int32_t* tok_pos, PagedKV kp, PagedKV vp, int n_tokens, int n_heads,
                           int maps, float scale, const float* head_scale, int window, int chunk, PooledKV pooled,
-                          const float* gate, long ldg, int gate_per, float softcap, cudaStream_t stream) {
+                          const float* gate, long ldg, int gate_per, float softcap, const float* r1, const float* r2,
+                          const float* sink, cudaStream_t stream) {
   const long items = (long)n_tokens * n_heads * maps;
   const long blocks = (items + FLEX_WARPS - 1) / FLEX_WARPS;
   if (blocks > 0x7fffffffL) return LLMI_ERR_BAD_SIZE;
@@ -264,7 +271,8 @@ int launch_attention_flex(const void* q, long ldq, void* out, long ldo, const vo
 #define LLMI_LAUNCH(NJ)                                                                                                  \
   return launch_pdl(PDL_ATTENTION, attention_flex_kernel<T, OutT, NJ>, dim3((unsigned)blocks), dim3(FLEX_WARPS * 32), 0, \
                     stream, (const T*)q, ldq, (OutT*)out, ldo, (const T*)k_cache, (const T*)v_cache, tok_seq, tok_pos,   \
-                    kp, vp, n_tokens, n_heads, maps, scale, head_scale, window, chunk, pooled, gate, ldg, gate_per, softcap)
+                    kp, vp, n_tokens, n_heads, maps, scale, head_scale, window, chunk, pooled, gate, ldg, gate_per, softcap, \
+                    r1, r2, sink)
   if (nj <= 1) LLMI_LAUNCH(1);
   if (nj <= 2) LLMI_LAUNCH(2);
   if (nj <= 4) LLMI_LAUNCH(4);
@@ -312,17 +320,18 @@ LLMI_EXPORT int llmi_attention_flex(int dtype, const void* q, long ldq, void* ou
                                     int n_kv_heads, int maps, int dk, int dv, float scale, const float* head_scale, int window,
                                     int chunk, int pool, const void* k_pool, const void* v_pool, const int32_t* pool_pages,
                                     int pool_pages_stride, const float* gate, long ldg, int gate_per, float softcap,
-                                    cudaStream_t stream) {
+                                    const float* r1, const float* r2, const float* sink, cudaStream_t stream) {
   if (n_tokens <= 0 || n_heads <= 0 || n_kv_heads <= 0 || maps <= 0 || dk <= 0 || dv <= 0 || page_size <= 0) return LLMI_ERR_BAD_SIZE;
   if (gate && gate_per != 1 && (gate_per != dv || maps != 1)) return LLMI_ERR_UNSUPPORTED;
-  if (softcap < 0.f) return LLMI_ERR_BAD_SIZE;
+  if (softcap < 0.f || (r1 == nullptr) != (r2 == nullptr)) return LLMI_ERR_BAD_SIZE;
+  if (r1 && pool > 0) return LLMI_ERR_UNSUPPORTED;          // a pooled row has no distance
   if (dk > FLEX_MAX_DK || dv > FLEX_MAX_DV || n_heads % n_kv_heads != 0 || window < 0 || chunk < 0) return LLMI_ERR_BAD_SIZE;
   if (pool < 0 || (pool > 0 && (!k_pool || !v_pool || !pool_pages || window <= 0))) return LLMI_ERR_BAD_SIZE;
   const PagedKV kp{seq_pages, pages_stride, page_size, n_kv_heads * maps, dk}, vp{seq_pages, pages_stride, page_size, n_kv_heads, dv};
   PooledKV pooled{pool > 0 ? k_pool : nullptr, pool > 0 ? v_pool : nullptr,
                   PagedKV{pool_pages, pool_pages_stride, page_size, n_kv_heads * maps, dk},
                   PagedKV{pool_pages, pool_pages_stride, page_size, n_kv_heads, dv}, pool};
-#define LLMI_ARGS q, ldq, out, ldo, k_cache, v_cache, tok_seq, tok_pos, kp, vp, n_tokens, n_heads, maps, scale, head_scale, window, chunk, pooled, gate, ldg, gate_per, softcap, stream
+#define LLMI_ARGS q, ldq, out, ldo, k_cache, v_cache, tok_seq, tok_pos, kp, vp, n_tokens, n_heads, maps, scale, head_scale, window, chunk, pooled, gate, ldg, gate_per, softcap, r1, r2, sink, stream
   if (dtype == LLMI_DTYPE_F32) return launch_attention_flex<float, float>(LLMI_ARGS);
   if (dtype == LLMI_DTYPE_BF16)
     return out_f32 ? launch_attention_flex<__nv_bfloat16, float>(LLMI_ARGS) : launch_attention_flex<__nv_bfloat16, __nv_bfloat16>(LLMI_ARGS);

@@ -23,6 +23,9 @@
 // the window's pages in the same loop and the same running softmax; and optionally every head's output is multiplied by
 // the logistic function of a number per (token, head), or every output entry by that of a number of its own; and
 // optionally (softcap > 0) a score passes softcap * tanh(score / softcap) before the softmax.
+// With `r1` and `r2` (a number per head each) a key d positions back loses r1 * ln(1 + r2 * d) of its score; a prompt's warp
+// makes the values for the distances of its 16 rows to a page's 64 keys once per page (79 of them, in shared memory)
+// instead of once per score.  With `sink` (a number per head) exp(sink) joins the softmax's sum and stands for no key.
 // The order of every addition depends on positions only (pages anchored at multiples of 64, parts by key index), not
 // on the batch; cuts follow the page table's width, which is part of a recorded step's shape.
 #include <math.h>
@@ -70,6 +73,9 @@ struct MapsArgs {
   long ldg;
   int gate_per;                 // 1: a number per head; dv: a number per output entry, at gate[t * ldg + h * dv + d] (one map)
   float softcap_log2;           // softcap * log2(e); 0: scores are not capped
+  const float* r1;              // [H] or null: the bias by distance (in base 2: r1 * log2(1 + r2 * d))
+  const float* r2;
+  const float* sink;            // [H] or null
 };
 
 __device__ __forceinline__ int maps_pooled_visible(int pos, int window, int pool) {
@@ -82,11 +88,18 @@ __device__ __forceinline__ float maps_gate(const MapsArgs& a, int t, int head) {
 __device__ __forceinline__ float maps_gate_entry(const MapsArgs& a, int t, int head, int dv, int d) {
   return (a.gate && a.gate_per > 1) ? 1.0f / (1.0f + __expf(-a.gate[(size_t)t * a.ldg + (size_t)head * dv + d])) : 1.0f;
 }
+// exp(sink) relative to the row's maximum m (base 2): what the sink adds to the softmax's sum.  (A sink far above every
+// score gives infinity, and the output is 0.)
+__device__ __forceinline__ float maps_sink(const float* sink, int head, float m) {
+  return sink ? exp2f(sink[head] * 1.4426950408889634f - m) : 0.f;
+}
 // tanh on the exponential unit: 1 - 2 / (1 + e^(2x)); x is a score over its cap, the result ends up in a bf16 weight
 __device__ __forceinline__ float maps_tanh(float x) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x)); }
 
-// NV = dv / 16.  PROMPT: the form (see above).
-template <int NV, bool PROMPT>
+constexpr int AM_BIAS = 80;      // distances of 16 rows to 64 keys: 79
+
+// NV = dv / 16.  PROMPT: the form (see above).  BIAS: with a bias by distance.
+template <int NV, bool PROMPT, bool BIAS>
 __global__ void __launch_bounds__((PROMPT ? AM_PROMPT_WARPS : AM_WARPS) * 32)
 attention_maps_mma_kernel(const MapsArgs a) {
   extern __shared__ __align__(16) unsigned char am_smem[];
@@ -94,6 +107,7 @@ attention_maps_mma_kernel(const MapsArgs a) {
   pdl_launch_dependents();
   constexpr int DV = NV * 16, ROWS = PROMPT ? AM_PROMPT_ROWS : 16, NT2 = PROMPT ? 4 : 1;
   constexpr int NBUF = PROMPT ? 2 : AM_TOKEN_BUFFERS;             // page buffers: NBUF - 1 pages are under way while one is multiplied     // NT2: groups of 16 keys a warp takes per page
+  __shared__ float bias_s[BIAS && PROMPT ? AM_PROMPT_WARPS * AM_BIAS : 1];
   const int dk = a.dk, ldk = dk + AM_PAD, ldv = DV + AM_PAD;
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(am_smem);                // [ROWS][ldk]
   __nv_bfloat16* k_s = q_s + ROWS * ldk;                                          // [NBUF][64][ldk]
@@ -156,7 +170,7 @@ attention_maps_mma_kernel(const MapsArgs a) {
 
   // my two rows (g and g + 8 of my warp's 16): position, first visible key, pooled blocks it sees, factor on the scores
   int row_pos[2], row_lo[2], row_nb[2];
-  float row_scale[2];
+  float row_scale[2], row_r1[2], row_r2[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = (PROMPT ? 16 * warp : 0) + g + 8 * i;
@@ -166,6 +180,8 @@ attention_maps_mma_kernel(const MapsArgs a) {
     row_nb[i] = ok ? maps_pooled_visible(row_pos[i], a.window, a.pool) : 0;
     const int head = PROMPT ? head0 : head0 + (ok ? r : 0);
     row_scale[i] = a.head_scale ? a.scale_log2 * a.head_scale[head] : a.scale_log2;
+    row_r1[i] = BIAS ? a.r1[head] : 0.f;
+    row_r2[i] = BIAS ? a.r2[head] : 0.f;
   }
   // what my warp's rows can see at all (a page outside costs my warp nothing)
   int w_hi, w_lo;
@@ -268,6 +284,14 @@ attention_maps_mma_kernel(const MapsArgs a) {
         mma_bf16(s[2 * c + 1], af, bf[2], bf[3]);
       }
     }
+    // the bias for every distance of my warp's rows to this page's keys, from that of the first row to the last key on
+    float* bias_w = bias_s + (BIAS && PROMPT ? warp * AM_BIAS : 0);
+    if (BIAS && PROMPT) {
+      __syncwarp();                                              // the page before is read out
+      const int d0 = p_first + 16 * warp - (base + AM_PAGE - 1);
+      for (int i = lane; i < AM_BIAS - 1; i += 32) bias_w[i] = row_r1[0] * fast_log2(fmaf(row_r2[0], (float)max(d0 + i, 0), 1.0f));
+      __syncwarp();
+    }
     // scale, mask, and the maximum of each of my rows over my keys
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -278,6 +302,8 @@ attention_maps_mma_kernel(const MapsArgs a) {
         const bool seen = pooled ? key < row_nb[i] : (key <= row_pos[i] && key >= row_lo[i]);
         float v = seen ? s[j][e] * row_scale[i] : -INFINITY;
         if (a.softcap_log2 > 0.f && seen) v = a.softcap_log2 * maps_tanh(v * inv_cap);
+        if (BIAS && PROMPT) v -= bias_w[g + 8 * i + AM_PAGE - 1 - (8 * j + 2 * tq + (e & 1))];
+        if (BIAS && !PROMPT) v -= row_r1[i] * fast_log2(fmaf(row_r2[i], (float)max(row_pos[i] - key, 0), 1.0f));
         s[j][e] = v;
         mx[i] = fmaxf(mx[i], v);
       }
@@ -332,7 +358,7 @@ attention_maps_mma_kernel(const MapsArgs a) {
     if (!PROMPT || row_pos[i] < 0) continue;
     {
       const int t = t0 + 16 * warp + g + 8 * i;
-      const float inv = maps_gate(a, t, head0) / l_run[i];
+      const float inv = maps_gate(a, t, head0) / (l_run[i] + maps_sink(a.sink, head0, m_run[i]));
       const size_t at = (size_t)t * a.ldo + (size_t)(head0 * a.maps + mp) * DV + 2 * tq;
 #pragma unroll
       for (int j = 0; j < 2 * NV; ++j) {
@@ -376,7 +402,7 @@ attention_maps_mma_kernel(const MapsArgs a) {
       const size_t hm = (size_t)(head0 + r) * a.maps + mp;
       if (a.splits == 1) {
         const size_t at = (size_t)t0 * a.ldo + hm * DV + c;
-        const float res = acc / l * maps_gate(a, t0, head0 + r) * maps_gate_entry(a, t0, head0 + r, DV, c);
+        const float res = acc / (l + maps_sink(a.sink, head0 + r, M)) * maps_gate(a, t0, head0 + r) * maps_gate_entry(a, t0, head0 + r, DV, c);
         if (a.out_f32) ((float*)a.out)[at] = res;
         else ((__nv_bfloat16*)a.out)[at] = __float2bfloat16_rn(res);
       } else {
@@ -396,7 +422,7 @@ constexpr int AM_MAX_PARTS = 1024;
 __global__ void __launch_bounds__(128)
 attention_maps_join_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml, void* __restrict__ out, long ldo,
                            int out_f32, const int32_t* __restrict__ tok_seq, int per_tok, int dv, int parts,
-                           const float* __restrict__ gate, long ldg, int maps, int gate_per) {
+                           const float* __restrict__ gate, long ldg, int maps, int gate_per, const float* __restrict__ sink) {
   __shared__ float w_s[AM_MAX_PARTS];
   __shared__ float red[32];
   pdl_wait();
@@ -421,7 +447,7 @@ attention_maps_join_kernel(const float* __restrict__ ws_o, const float* __restri
     w_s[s] = w;
     part += w * ml[2 * s + 1];
   }
-  float inv = 1.0f / block_sum(part, red);
+  float inv = 1.0f / (block_sum(part, red) + maps_sink(sink, hm / maps, M));
   if (gate && gate_per <= 1) inv *= 1.0f / (1.0f + __expf(-gate[(size_t)t * ldg + hm / maps]));
   const float* o = ws_o + (size_t)item * parts * dv;
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
@@ -435,16 +461,20 @@ attention_maps_join_kernel(const float* __restrict__ ws_o, const float* __restri
   }
 }
 
-template <int NV, bool PROMPT>
-int launch_maps_mma(const MapsArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+template <int NV, bool PROMPT, bool BIAS>
+int launch_maps_mma_b(const MapsArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
   static PerDevice<size_t> allowed;
   if (smem > 48 * 1024 && allowed.here() < smem) {
-    if (cudaFuncSetAttribute(attention_maps_mma_kernel<NV, PROMPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_maps_mma_kernel<NV, PROMPT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return LLMI_ERR_BAD_SIZE;
     allowed.here() = smem;
   }
-  return launch_pdl(PDL_ATTENTION, attention_maps_mma_kernel<NV, PROMPT>, grid, dim3((PROMPT ? AM_PROMPT_WARPS : AM_WARPS) * 32), smem,
+  return launch_pdl(PDL_ATTENTION, attention_maps_mma_kernel<NV, PROMPT, BIAS>, grid, dim3((PROMPT ? AM_PROMPT_WARPS : AM_WARPS) * 32), smem,
                     stream, a);
+}
+template <int NV, bool PROMPT>
+int launch_maps_mma(const MapsArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+  return a.r1 ? launch_maps_mma_b<NV, PROMPT, true>(a, grid, smem, stream) : launch_maps_mma_b<NV, PROMPT, false>(a, grid, smem, stream);
 }
 
 }  // namespace llmi
@@ -472,9 +502,10 @@ LLMI_EXPORT int llmi_attention_maps_mma(const void* q, long ldq, void* out, long
                                         int n_blocks, int splits, int pages_per_split, float* workspace, long workspace_floats,
                                         int pool, const void* k_pool, const void* v_pool, const int32_t* pool_pages,
                                         int pool_pages_stride, const float* gate, long ldg, int gate_per, float softcap,
-                                        cudaStream_t stream) {
+                                        const float* r1, const float* r2, const float* sink, cudaStream_t stream) {
   if (gate && gate_per != 1 && (gate_per != dv || maps != 1)) return LLMI_ERR_UNSUPPORTED;
-  if (softcap < 0.f) return LLMI_ERR_BAD_SIZE;
+  if (softcap < 0.f || (r1 == nullptr) != (r2 == nullptr)) return LLMI_ERR_BAD_SIZE;
+  if (r1 && pool > 0) return LLMI_ERR_UNSUPPORTED;          // a pooled row has no distance
   if (n_tokens <= 0 || n_seqs <= 0 || n_heads <= 0 || n_kv_heads <= 0 || maps <= 0 || n_heads % n_kv_heads) return LLMI_ERR_BAD_SIZE;
   if (!llmi_attention_maps_mma_supported(dk, dv, n_heads / n_kv_heads, AM_PAGE)) return LLMI_ERR_UNSUPPORTED;
   if (((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15) || (ldq % 8) || ((uintptr_t)out & 7) || (ldo % 2))
@@ -492,6 +523,7 @@ LLMI_EXPORT int llmi_attention_maps_mma(const void* q, long ldq, void* out, long
   a.pool = pool; a.k_pool = (const __nv_bfloat16*)k_pool; a.v_pool = (const __nv_bfloat16*)v_pool;
   a.pool_pages = pool_pages; a.pool_pages_stride = pool_pages_stride; a.gate = gate; a.ldg = ldg;
   a.gate_per = gate_per; a.softcap_log2 = softcap * 1.4426950408889634f;
+  a.r1 = r1; a.r2 = r2; a.sink = sink;
   const int rows = prompt ? AM_PROMPT_ROWS : 16;
   const int nbuf = prompt ? 2 : AM_TOKEN_BUFFERS;
   const size_t smem = ((size_t)(rows + nbuf * AM_PAGE) * (dk + AM_PAD) + (size_t)nbuf * AM_PAGE * (dv + AM_PAD)) * 2;
@@ -519,5 +551,5 @@ LLMI_EXPORT int llmi_attention_maps_mma(const void* q, long ldq, void* out, long
   const long items = (long)n_tokens * n_heads * maps;
   if (items > 0x7fffffffL) return LLMI_ERR_BAD_SIZE;
   return launch_pdl(PDL_SMALL, attention_maps_join_kernel, dim3((unsigned)items), dim3(128), 0, stream, (const float*)a.ws_o,
-                    (const float*)a.ws_ml, out, ldo, out_f32, tok_seq, n_heads * maps, dv, splits, gate, ldg, maps, gate_per);
+                    (const float*)a.ws_ml, out, ldo, out_f32, tok_seq, n_heads * maps, dv, splits, gate, ldg, maps, gate_per, sink);
 }

@@ -23,6 +23,10 @@
 // read-multiply-write of O in TMEM happens a few times per row instead of once per page (only then is
 // O += P_{j-1} V_{j-1} waited for); the final division by the row sum makes the result the same.
 //
+// Optionally a key d positions back loses r1[h] * ln(1 + r2[h] * d) of its score: a softmax warp makes the values for the
+// distances of its 32 rows to its keys of a page (63 or 95 of them) once per page in shared memory, two or three a lane,
+// and every score then costs one shared-memory read instead of a logarithm.  Optionally exp(sink[h]) joins a head's sum.
+//
 // A causal prompt's query blocks differ 16-fold in the keys they see, and the kernel is as long as its longest
 // block: with `split_pages` > 0 a block's key range is cut into parts of that many pages, each part a block of
 // its own that leaves (reference maximum, sum, unnormalised output) per row in a workspace; the part that takes
@@ -85,6 +89,9 @@ struct PrefillTcParams {
   int pool_pages_stride;
   const float* gate;        // [tokens, >= n_heads] fp32 or null: head h's output times logistic(gate[t, h])
   long ldg;
+  const float* r1;          // [n_heads] fp32 or null: the bias by distance (base 2: r1 * log2(1 + r2 * d))
+  const float* r2;
+  const float* sink;        // [n_heads] fp32 or null
 };
 
 __device__ __forceinline__ void ft_tma(uint32_t dst, const CUtensorMap* map, int col, int row, uint32_t bar) {
@@ -149,7 +156,7 @@ __device__ __forceinline__ void ft_st16u(uint32_t taddr, const uint32_t* v) {
       : "memory");
 }
 
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __launch_bounds__(FtCfg<HD>::THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_kp,
@@ -221,6 +228,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const int kvh = head / (p.n_heads / p.n_kv_heads);
   const int32_t* pages = p.seq_pages + (size_t)seq * p.pages_stride;
   __shared__ int s_last;
+  __shared__ float bias_s[BIAS ? 4 * HALVES * (31 + KEYS + 1) : 1];
   __shared__ float s_ml[2][FT_BM][2];      // (reference maximum, sum) of a row's two key halves
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -342,6 +350,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const uint32_t t_lane = (uint32_t)(quad * 32) << 16;
     const uint32_t t_o = tmem_o + t_lane + (uint32_t)(HD * half);
     float m_run = -INFINITY, m_ref = -INFINITY, l_run = 0.f;   // maxima in base 2, scaled
+    float* bias_w = bias_s + (BIAS ? (warp - 2) * (31 + KEYS + 1) : 0);
+    const float r1 = BIAS ? p.r1[head] : 0.f, r2 = BIAS ? p.r2[head] : 0.f;      // (weights: no kernel before writes them)
     bool ok = true;
     for (int j = 0; j < n_pg && ok; ++j) {
       ok = mbar_wait(s_full(j & 1), (j >> 1) & 1, p.error_flag, 48);
@@ -369,6 +379,21 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           if (key > qpos || (p.window > 0 && key < qpos - p.window + 1)) sc[c] = -INFINITY;
         }
       }
+      if (BIAS) {
+        // distances from my warp's first row to its last key of the page on; then scores are base 2 and final
+        __syncwarp();                                                   // the page before is read out
+        const int d0 = pos0 + m0 + quad * 32 - (key0 + KEYS - 1);
+#pragma unroll
+        for (int i = 0; i < KEYS / 32 + 1; ++i) {
+          const int e = lane + 32 * i;
+          bias_w[e] = r1 * fast_log2(fmaf(r2, (float)max(d0 + e, 0), 1.0f));
+        }
+        __syncwarp();
+        const float* bias_l = bias_w + lane + KEYS - 1;
+#pragma unroll
+        for (int c = 0; c < KEYS; ++c) sc[c] = fmaf(sc[c], p.scale_log2, -bias_l[-c]);
+      }
+      const float to_log2 = BIAS ? 1.0f : p.scale_log2;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains instead of one long one
 #pragma unroll
       for (int c = 0; c < KEYS; c += 8) {
@@ -376,7 +401,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         for (int u = 0; u < 4; ++u) mx4[u] = fmaxf(mx4[u], fmaxf(sc[c + 2 * u], sc[c + 2 * u + 1]));
       }
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      m_run = fmaxf(m_run, mx * p.scale_log2);
+      m_run = fmaxf(m_run, mx * to_log2);
       float corr = 1.f;
       if (m_run > m_ref + FT_LAZY || m_ref == -INFINITY) {     // (both -inf: nothing seen yet, nothing to scale)
         corr = (m_ref == -INFINITY) ? 0.f : fast_exp2(m_ref - m_run);
@@ -386,7 +411,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const float neg_ref = (m_ref == -INFINITY) ? 0.f : -m_ref;
       // two keys per instruction where the hardware has it (fma.rn.f32x2, add.rn.f32x2)
       float2 sum2[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};
-      const float2 scale2 = make_float2(p.scale_log2, p.scale_log2), neg2 = make_float2(neg_ref, neg_ref);
+      const float2 scale2 = make_float2(to_log2, to_log2), neg2 = make_float2(neg_ref, neg_ref);
       uint32_t packed[KEYS / 2];
 #pragma unroll
       for (int c = 0; c < KEYS; c += 2) {
@@ -508,7 +533,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
       }
       if (write_out) {      // every lane takes part in the TMEM loads; only the rows that exist are stored
-        float inv = 1.f / L;
+        float inv = 1.f / (p.sink ? L + fast_exp2(p.sink[head] * 1.4426950408889634f - M) : L);
         if (p.gate && row_ok) inv *= 1.0f / (1.0f + expf(-p.gate[(size_t)(q_start + qrow) * p.ldg + head]));
         __nv_bfloat16* dst = p.out + (size_t)(q_start + qrow) * p.ldo + (size_t)head * HD + DH * half;
 #pragma unroll 1
@@ -592,20 +617,25 @@ using namespace llmi;
 LLMI_EXPORT int llmi_attention_prefill_tc_supported(int head_dim) { return head_dim == 64 || head_dim == 128; }
 
 namespace llmi {
-template <int HD>
-static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkp,
+template <int HD, bool BIAS>
+static int ft_launch_b(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkp,
                      const CUtensorMap& mvp, const PrefillTcParams& p, dim3 grid, cudaStream_t stream) {
   using C = FtCfg<HD>;
   static PerDevice<bool> configured_on;
   bool& configured = configured_on.here();
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) != cudaSuccess)
       return LLMI_ERR_LAUNCH;
     configured = true;
   }
   // a programmatic dependent: its blocks set themselves up (barriers, tensor memory, descriptors) while the kernel
   // before drains; the producer waits before its first copy, and nothing else reads or writes global memory earlier
-  return launch_pdl(PDL_ATTENTION, attention_prefill_tc_kernel<HD>, grid, dim3(C::THREADS), C::SMEM, stream, mq, mk, mv, mkp, mvp, p);
+  return launch_pdl(PDL_ATTENTION, attention_prefill_tc_kernel<HD, BIAS>, grid, dim3(C::THREADS), C::SMEM, stream, mq, mk, mv, mkp, mvp, p);
+}
+template <int HD>
+static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkp,
+                     const CUtensorMap& mvp, const PrefillTcParams& p, dim3 grid, cudaStream_t stream) {
+  return p.r1 ? ft_launch_b<HD, true>(mq, mk, mv, mkp, mvp, p, grid, stream) : ft_launch_b<HD, false>(mq, mk, mv, mkp, mvp, p, grid, stream);
 }
 }  // namespace llmi
 
@@ -613,7 +643,9 @@ static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 // pool > 0 (with a window): one pooled key and value row per block of `pool` positions that lies wholly before a
 // query's window, in k_pool / v_pool [n_pool_cache_pages, n_kv_heads, 64, head_dim] under the page table pool_pages
 // [n_seqs, pool_pages_stride] (row b of a sequence's pooled pages is block b); they share the softmax with the window's
-// keys.  gate (optional): fp32 [n_tokens, ldg], head h's output is multiplied by logistic(gate[t, h]).
+// keys.  gate (optional): fp32 [n_tokens, ldg], head h's output is multiplied by logistic(gate[t, h]).  r1, r2 (optional, not
+// with pooled rows): fp32 [n_heads], a key d positions back loses r1 * ln(1 + r2 * d) of its score; sink (optional): fp32
+// [n_heads], exp(sink) joins the head's softmax sum.
 // With split_pages > 0: partials holds n_jobs * n_heads * (head_dim + 2) * 128 floats.
 LLMI_EXPORT int llmi_attention_prefill_tc(const void* q, long ldq, long n_tokens, void* out, long ldo, const void* k_cache,
                                           const void* v_cache, long n_cache_pages, const int32_t* seq_pages,
@@ -622,10 +654,13 @@ LLMI_EXPORT int llmi_attention_prefill_tc(const void* q, long ldq, long n_tokens
                                           int window, int n_jobs, int split_pages, float* partials, long partials_floats,
                                           int* tickets, int n_tickets, int* error_flag, int pool, const void* k_pool,
                                           const void* v_pool, long n_pool_cache_pages, const int32_t* pool_pages,
-                                          int pool_pages_stride, const float* gate, long ldg, cudaStream_t stream) {
+                                          int pool_pages_stride, const float* gate, long ldg, const float* r1, const float* r2,
+                                          const float* sink, cudaStream_t stream) {
   if (n_seqs <= 0 || n_blocks <= 0 || n_heads <= 0 || n_kv_heads <= 0 || n_cache_pages <= 0 || n_tokens <= 0) return LLMI_ERR_BAD_SIZE;
   if (n_heads % n_kv_heads) return LLMI_ERR_BAD_SIZE;
   if (!llmi_attention_prefill_tc_supported(head_dim)) return LLMI_ERR_UNSUPPORTED;
+  if ((r1 == nullptr) != (r2 == nullptr) || (r1 && scale <= 0.f)) return LLMI_ERR_BAD_SIZE;
+  if (r1 && pool > 0) return LLMI_ERR_UNSUPPORTED;            // a pooled row has no distance
   if (((uintptr_t)q & 15) || (ldq & 7) || ((uintptr_t)out & 15) || (ldo & 7) || ((uintptr_t)k_cache & 15) ||
       ((uintptr_t)v_cache & 15))
     return LLMI_ERR_ALIGN;
@@ -663,7 +698,7 @@ LLMI_EXPORT int llmi_attention_prefill_tc(const void* q, long ldq, long n_tokens
   }
   PrefillTcParams p{(__nv_bfloat16*)out, ldo, seq_pages, seq_q_start, seq_kv_len, pages_stride, n_seqs, n_heads,
                     n_kv_heads, scale * 1.4426950408889634f, window, error_flag, n_blocks, split_pages, partials, tickets,
-                    pool, pool_pages, pool_pages_stride, gate, ldg};
+                    pool, pool_pages, pool_pages_stride, gate, ldg, r1, r2, sink};
   if (n_jobs > 65535) return LLMI_ERR_BAD_SIZE;
   dim3 grid(n_heads, n_jobs);
   return head_dim == 64 ? ft_launch<64>(mq, mk, mv, mkp, mvp, p, grid, stream) : ft_launch<128>(mq, mk, mv, mkp, mvp, p, grid, stream);

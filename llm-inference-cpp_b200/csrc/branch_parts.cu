@@ -3,6 +3,10 @@
 //                          normed over the model width with a weight of its own, then averaged (c = 1/2)
 //   llmi_stream_axpy_norm  x[t] += m * y[t], and (optionally) h[t] = norm_w * x[t] / rms(x[t]) of the new x in the same
 //                          pass: the norm ahead of the next layer
+//   llmi_stream_postnorm   x[t] = norm_w * v / rms(v) with v = a * x[t] + y[t]: a branch joins the stream and the norm BEHIND
+//                          the sum replaces it; h[t] receives the new x in the compute type (what the next branch reads).
+//                          Without y and norm_w: only the copy h = x
+//   llmi_softcap_rows      v = cap * tanh(v / cap) in place (the logits)
 // rms(v) = sqrt(mean(v^2) + eps).  All arithmetic fp32; a block per row, rows are treated alone.
 #include <math.h>
 
@@ -109,6 +113,74 @@ stream_axpy_norm_kernel(float* __restrict__ x, const float* __restrict__ y, floa
   }
 }
 
+// Each thread keeps its pieces of the row in registers (up to PN_KEEP of them; what is left is formed twice).
+constexpr int PN_KEEP = 4;
+template <typename T>
+__global__ void __launch_bounds__(512)
+stream_postnorm_kernel(float* __restrict__ x, const float* __restrict__ y, float alpha, int W, const float* __restrict__ norm_w,
+                       float eps, T* __restrict__ h) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  float* xr = x + (size_t)t * W;
+  const float* yr = y ? y + (size_t)t * W : nullptr;
+  T* hr = h ? h + (size_t)t * W : nullptr;
+  if (!y) {
+    for (int i = threadIdx.x; i < W; i += blockDim.x) hr[i] = from_f32<T>(xr[i]);
+    return;
+  }
+  float ss = 0.f;
+  if (W % 4 == 0) {
+    auto joined = [&](int i) {
+      const float4 v = reinterpret_cast<const float4*>(xr)[i], u = reinterpret_cast<const float4*>(yr)[i];
+      return make_float4(fmaf(alpha, v.x, u.x), fmaf(alpha, v.y, u.y), fmaf(alpha, v.z, u.z), fmaf(alpha, v.w, u.w));
+    };
+    float4 keep[PN_KEEP];
+#pragma unroll
+    for (int k = 0; k < PN_KEEP; ++k) {
+      const int i = threadIdx.x + k * blockDim.x;
+      keep[k] = i < W / 4 ? joined(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss = fmaf(keep[k].x, keep[k].x, ss); ss = fmaf(keep[k].y, keep[k].y, ss);
+      ss = fmaf(keep[k].z, keep[k].z, ss); ss = fmaf(keep[k].w, keep[k].w, ss);
+    }
+    for (int i = threadIdx.x + PN_KEEP * blockDim.x; i < W / 4; i += blockDim.x) {
+      const float4 v = joined(i);
+      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+    }
+    const float scale = 1.0f / sqrtf(block_sum(ss, scratch) / (float)W + eps);
+    auto leave = [&](int i, float4 v) {
+      const float4 w = reinterpret_cast<const float4*>(norm_w)[i];
+      v = make_float4(w.x * (v.x * scale), w.y * (v.y * scale), w.z * (v.z * scale), w.w * (v.w * scale));
+      reinterpret_cast<float4*>(xr)[i] = v;
+      if (hr) store4(hr + 4 * i, v.x, v.y, v.z, v.w);
+    };
+#pragma unroll
+    for (int k = 0; k < PN_KEEP; ++k) {
+      const int i = threadIdx.x + k * blockDim.x;
+      if (i < W / 4) leave(i, keep[k]);
+    }
+    for (int i = threadIdx.x + PN_KEEP * blockDim.x; i < W / 4; i += blockDim.x) leave(i, joined(i));
+  } else {
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+      const float v = fmaf(alpha, xr[i], yr[i]);
+      ss = fmaf(v, v, ss);
+    }
+    const float scale = 1.0f / sqrtf(block_sum(ss, scratch) / (float)W + eps);
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+      const float v = norm_w[i] * (fmaf(alpha, xr[i], yr[i]) * scale);
+      xr[i] = v;
+      if (hr) hr[i] = from_f32<T>(v);
+    }
+  }
+}
+
+__global__ void __launch_bounds__(256) softcap_rows_kernel(float* __restrict__ v, size_t n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) v[i] = cap * tanhf(v[i] / cap);
+}
+
 }  // namespace llmi
 
 using namespace llmi;
@@ -138,4 +210,27 @@ LLMI_EXPORT int llmi_stream_axpy_norm(float* x, const float* y, float m, int n_r
     return launch_pdl(PDL_SMALL, stream_axpy_norm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, stream, x, y, m, W, norm_w,
                       eps, (__nv_bfloat16*)h);
   return LLMI_ERR_BAD_DTYPE;
+}
+
+// x, y fp32 [T, W] contiguous; norm_w fp32 [W]; h [T, W] contiguous in `dtype`, or null.  x = norm_w * v / rms(v) with
+// v = alpha * x + y, and h = x; with y null only h = x.
+LLMI_EXPORT int llmi_stream_postnorm(float* x, const float* y, float alpha, int n_rows, int W, const float* norm_w, float eps, int dtype,
+                                     void* h, cudaStream_t stream) {
+  if (n_rows <= 0 || W <= 0 || (y == nullptr) != (norm_w == nullptr) || (!y && !h)) return LLMI_ERR_BAD_SIZE;
+  if (W % 4 == 0 && (((uintptr_t)x & 15) || ((uintptr_t)y & 15) || ((uintptr_t)norm_w & 15) || ((uintptr_t)h & 15))) return LLMI_ERR_ALIGN;
+  const int threads = W >= 2048 ? 512 : (W >= 1024 ? 256 : (W >= 256 ? 128 : 64));
+  if (!h || dtype == LLMI_DTYPE_F32)
+    return launch_pdl(PDL_SMALL, stream_postnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, x, y, alpha, W, norm_w, eps,
+                      (float*)h);
+  if (dtype == LLMI_DTYPE_BF16)
+    return launch_pdl(PDL_SMALL, stream_postnorm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, stream, x, y, alpha, W, norm_w,
+                      eps, (__nv_bfloat16*)h);
+  return LLMI_ERR_BAD_DTYPE;
+}
+
+// v fp32, n entries: v = cap * tanh(v / cap) in place.
+LLMI_EXPORT int llmi_softcap_rows(float* v, long n, float cap, cudaStream_t stream) {
+  if (n <= 0 || !(cap > 0.f)) return LLMI_ERR_BAD_SIZE;
+  const long most = (long)sm_count() * 8, need = (n + 255) / 256;
+  return launch_pdl(PDL_SMALL, softcap_rows_kernel, dim3((unsigned)(need < most ? need : most)), dim3(256), 0, stream, v, (size_t)n, cap);
 }

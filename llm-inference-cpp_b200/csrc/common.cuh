@@ -69,6 +69,13 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// log2(x) on the special-function unit, one instruction (lg2.approx: absolute error about 2^-22 near 1, relative elsewhere).
+__device__ __forceinline__ float fast_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // The rotation of one pair, with its roundings spelled out so that every kernel that rotates gives the
 // same bits whatever the compiler would contract: the result must not depend on which kernel a step's
 // size selects.

@@ -7,7 +7,8 @@
 //     softmax     running maximum and sum per query row, fp32, shared by the four warps through shared memory
 //     O[16 x C]  += P[16 x 64] · rows[:, :C]      warp w: columns wC/4 .. (w+1)C/4 - 1; the page serves as key AND value
 // Pages arrive by cp.async into two buffers, the next one while the current one is multiplied; rows of a page beyond
-// the block's newest position arrive as zeros.  With `splits` > 1 (single tokens over long caches) grid.z cuts the
+// the block's newest position arrive as zeros.  With `window` > 0 a query sees the last `window` positions only: the walk
+// starts at the page of the block's oldest visible position.  With `splits` > 1 (single tokens over long caches) grid.z cuts the
 // positions; every cut leaves (maximum, sum, unnormalised O) in a workspace and a second kernel joins them.
 // Needs C % 64 == 0, (C + R) % 16 == 0, C <= 512, pages of 64 rows.
 #include <math.h>
@@ -36,6 +37,7 @@ struct LatentMmaArgs {
   int page_buffers;             // 2: the next page arrives while the current one is multiplied; 1: half the shared memory,
                                 // so that two blocks share an SM and overlap each other instead (steps of single tokens)
   float scale;
+  int window;                   // 0: every earlier position
   float* ws_o;                  // [T, H, splits, C]   (splits > 1)
   float* ws_ml;                 // [T, H, splits, 2]
 };
@@ -78,14 +80,15 @@ attention_latent_mma_kernel(const LatentMmaArgs a) {
   for (int seq = seq_lo; seq <= seq_hi; ++seq) {
     __syncthreads();                                           // the pass before has read q_s and k_s out
     // queries of this pass: rows of other sequences, of no token or of no head are zeros and see no key
-    int newest = -1;
+    int newest = -1, oldest = 0x7fffffff;
     for (int t = t0; t <= t_last; ++t)
-      if (a.tok_seq[t] == seq) newest = max(newest, a.tok_pos[t]);
-    int row_pos[2];
+      if (a.tok_seq[t] == seq) { newest = max(newest, a.tok_pos[t]); oldest = min(oldest, a.tok_pos[t]); }
+    int row_pos[2], row_lo[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const bool ok = row_tok[i] <= t_last && row_head[i] < a.n_heads && a.tok_seq[row_tok[i]] == seq;
       row_pos[i] = ok ? a.tok_pos[row_tok[i]] : -1;
+      row_lo[i] = ok ? first_visible(row_pos[i], a.window, 0) : 0;
     }
     const int chunks = Dk / 8;
     for (int idx = threadIdx.x; idx < RG * LM_ROWS * chunks; idx += blockDim.x) {
@@ -97,14 +100,15 @@ attention_latent_mma_kernel(const LatentMmaArgs a) {
       *reinterpret_cast<uint4*>(q_s + r * ldk + 8 * c8) = v;
     }
     const int n_pages = newest / LM_KEYS + 1;
-    const int pg_lo = split * a.pages_per_split, pg_hi = min(n_pages, pg_lo + a.pages_per_split);
+    const int first_key = newest < 0 ? 0 : first_visible(oldest, a.window, 0);
+    const int pg_lo = first_key / LM_KEYS + split * a.pages_per_split, pg_hi = min(n_pages, pg_lo + a.pages_per_split);
 
     auto fetch = [&](int pg, int buf) {
       const int page = a.seq_pages[(size_t)seq * a.pages_stride + pg];
       const __nv_bfloat16* src = a.cache + (size_t)page * LM_KEYS * Dk;
       __nv_bfloat16* dst = k_s + (size_t)buf * LM_KEYS * ldk;
       for (int r = threadIdx.x >> 5; r < LM_KEYS; r += RG * LM_WARPS) {          // a warp copies whole rows
-        const bool live = page >= 0 && pg * LM_KEYS + r <= newest;
+        const bool live = page >= 0 && pg * LM_KEYS + r <= newest && pg * LM_KEYS + r >= first_key;
         const __nv_bfloat16* from = live ? src + (size_t)r * Dk : a.cache;
         for (int c8 = lane; c8 < chunks; c8 += 32) cp_async16(dst + r * ldk + 8 * c8, live ? from + 8 * c8 : from, live ? 16 : 0);
       }
@@ -168,7 +172,7 @@ attention_latent_mma_kernel(const LatentMmaArgs a) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + 8 * j + (e & 1), i = e >> 1;
-          const float v = key <= row_pos[i] ? s[j][e] * a.scale : -INFINITY;
+          const float v = key <= row_pos[i] && key >= row_lo[i] ? s[j][e] * a.scale : -INFINITY;
           s[j][e] = v;
           mx[i] = fmaxf(mx[i], v);
         }
@@ -347,9 +351,9 @@ LLMI_EXPORT int llmi_attention_latent_mma(const void* qa, long ldq, void* out, l
                                           const int32_t* tok_seq, const int32_t* tok_pos, const int32_t* seq_pages,
                                           int pages_stride, int page_size, int n_tokens, int n_heads, int C, int R, float scale,
                                           int splits, int pages_per_split, int row_groups, float* workspace,
-                                          long workspace_floats, cudaStream_t stream) {
+                                          long workspace_floats, int window, cudaStream_t stream) {
   if (n_tokens <= 0 || n_heads <= 0 || !llmi_attention_latent_mma_supported(C, R, page_size)) return LLMI_ERR_UNSUPPORTED;
-  if (splits < 1 || splits > LM_MAX_SPLITS || pages_per_split < 1 || (row_groups != 1 && row_groups != 2)) return LLMI_ERR_BAD_SIZE;
+  if (splits < 1 || splits > LM_MAX_SPLITS || pages_per_split < 1 || (row_groups != 1 && row_groups != 2) || window < 0) return LLMI_ERR_BAD_SIZE;
   if (((uintptr_t)qa & 15) || ((uintptr_t)cache & 15) || (ldq % 8) || ((uintptr_t)out & 3) || (ldo % 2)) return LLMI_ERR_ALIGN;
   if (splits > 1 && (!workspace || workspace_floats < llmi_attention_latent_mma_workspace(n_tokens, n_heads, C, splits)))
     return LLMI_ERR_BAD_SIZE;
@@ -360,7 +364,7 @@ LLMI_EXPORT int llmi_attention_latent_mma(const void* qa, long ldq, void* out, l
   a.tok_seq = tok_seq; a.tok_pos = tok_pos; a.seq_pages = seq_pages; a.pages_stride = pages_stride;
   a.n_tokens = n_tokens; a.n_heads = n_heads; a.C = C; a.R = R;
   a.heads_per_block = hpb; a.tokens_per_block = row_groups * LM_ROWS / hpb;
-  a.splits = splits; a.pages_per_split = pages_per_split; a.scale = scale;
+  a.splits = splits; a.pages_per_split = pages_per_split; a.scale = scale; a.window = window;
   a.page_buffers = row_groups == 1 ? 1 : 2;
   a.ws_o = workspace;
   a.ws_ml = workspace ? workspace + (size_t)n_tokens * n_heads * splits * C : nullptr;

@@ -10,6 +10,7 @@
 //                     `n_identity` of the E router outputs stand for experts that hand their input on: such a choice
 //                     is written as index -1 (the product kernels skip it) and the token's summed weight of them to
 //                     `id_wt`, for llmi_moe_identity_add
+//   llmi_moe_table    per token: its experts from a table [vocab, top] by the token's id, each weighted 1 / top (no router)
 //   llmi_moe_up       per (token, choice): a = act(Wg_e h) * (Wu_e h), or a = act(Wu_e h) for experts
 //                     without a gate matrix                                                  [T, top, F] fp32
 //   llmi_moe_down     per token: y = sum over its choices, in the order of the choice, of weight * (Wd_e a)   [T, W] fp32
@@ -34,6 +35,20 @@ __device__ __forceinline__ void warp_best(float& best, int& best_e) {
     const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
     if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
   }
+}
+
+__global__ void __launch_bounds__(128)
+moe_table_kernel(const int32_t* __restrict__ table, int vocab, int top, const int32_t* __restrict__ token_ids,
+                 const int32_t* __restrict__ tok_seq, int32_t* __restrict__ idx, float* __restrict__ wt, int n_items) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n_items) return;
+  const int t = i / top, j = i - t * top;
+  const int id = token_ids[t];
+  const bool live = tok_seq[t] >= 0 && id >= 0 && id < vocab;
+  idx[i] = live ? table[(size_t)id * top + j] : -1;
+  wt[i] = live ? 1.0f / (float)top : 0.f;
 }
 
 // One warp per token.  MODE 0: softmax over the chosen logits.  MODE 1: logistic scores, normalised over the chosen.
@@ -274,6 +289,16 @@ LLMI_EXPORT int llmi_moe_route(const float* logits, long ld, int E, int top, int
                       idx, wt, n_tokens, correction, scale, n_identity, id_wt);
   }
   return LLMI_ERR_UNSUPPORTED;
+}
+
+// idx [T, top] = table[token_ids[t]] and wt [T, top] = 1 / top; a token row of no sequence gets index -1 and weight 0.
+LLMI_EXPORT int llmi_moe_table(const int32_t* table, int vocab, int top, const int32_t* token_ids, const int32_t* tok_seq, int32_t* idx,
+                               float* wt, int n_tokens, cudaStream_t stream) {
+  if (n_tokens <= 0 || vocab <= 0 || top <= 0) return LLMI_ERR_BAD_SIZE;
+  const long n = (long)n_tokens * top;
+  if (n > 0x7fffffffL) return LLMI_ERR_BAD_SIZE;
+  return launch_pdl(PDL_SMALL, moe_table_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, stream, table, vocab, top, token_ids,
+                    tok_seq, idx, wt, (int)n);
 }
 
 // y [T, ldy] fp32 += id_wt[t] * h[t] (h [T, ldh] in `dtype`).

@@ -10,6 +10,11 @@
 //   * q goes to `q_out` in the compute type; k and v go to the cache pages of (sequence, position).
 // Keys and values may differ in their number of heads and in their head size (two page layouts).  With `v_from_k`
 // the row has no v part: the values are the key rows as projected (after the norm, before the rotation), head for head.
+// A further form (qkv_unit_prepare) has no rotation and treats every head alone, a warp per (token, head):
+//   * q and k heads are divided by their root mean square over the head, sqrt(mean(x^2) + eps), no weight;
+//   * q is multiplied by a temperature that grows a step every `every` positions: 1 + coef * ln(floor((p + 1) / every) + 1);
+//   * v may be kept as it is for later layers (`v_first`, fp32), or mixed with what an earlier layer kept of the same
+//     token: (1 - lambda) v + lambda v_first; the mixed v is what the cache gets.
 // All arithmetic is fp32; one block per token, or, where no norm ties a part's heads together, one per (token, head).
 #include "common.cuh"
 #include "step_meta.cuh"
@@ -227,6 +232,120 @@ qkv_prepare_chunks_kernel(const float* __restrict__ proj, long ld, int n_q_heads
 }
 
 
+// VEC: four entries a lane and access (dk, dv, ld, ldq multiples of four and every base aligned to 16 bytes).
+constexpr int UP_WARPS = 4;
+struct UnitPrepareArgs {
+  const float* proj;            // [T, ld] = [ q: n_q * dk | k: n_k * dk | v: n_v * dv ]
+  long ld;
+  int n_q, n_k, dk, n_v, dv;
+  int unit;                     // 0: q and k heads stay as projected
+  float eps;
+  float temp_coef;
+  int temp_every;               // 0: no temperature
+  int v_mode;                   // 0: plain; 1: keep v in v_first; 2: mix with v_first
+  float lambda;
+  float* v_first;               // [T, n_v * dv]
+  const int32_t *tok_seq, *tok_pos;
+  PagedKV kp, vp;
+  long ldq;
+  int n_tokens, write_kv;
+};
+
+__device__ __forceinline__ void store4(float* o, const float4& v) { *reinterpret_cast<float4*>(o) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* o, const float4& v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const uint32_t*>(&lo);
+  u.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(o) = u;
+}
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(UP_WARPS * 32)
+qkv_unit_prepare_kernel(const UnitPrepareArgs a, T* __restrict__ k_cache, T* __restrict__ v_cache, T* __restrict__ q_out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n_all = a.n_q + a.n_k + a.n_v;
+  const long item = (long)blockIdx.x * UP_WARPS + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  const int t = (int)(item / n_all), hd = (int)(item - (long)t * n_all);
+  if (t >= a.n_tokens) return;
+  const int seq = a.tok_seq[t];
+  const float* row = a.proj + (size_t)t * a.ld;
+  if (hd < a.n_q + a.n_k) {
+    const bool is_q = hd < a.n_q;
+    const float* src = row + (size_t)hd * a.dk;
+    T* dst = q_out + (size_t)t * a.ldq + (size_t)hd * a.dk;
+    if (seq < 0) {
+      if (is_q)
+        for (int e = lane; e < a.dk; e += 32) dst[e] = from_f32<T>(0.f);
+      return;
+    }
+    const int pos = a.tok_pos[t];
+    if (!is_q) {
+      if (!a.write_kv) return;
+      dst = k_cache + kv_row_offset(a.kp, seq, pos, hd - a.n_q);
+    }
+    float sc = 1.f;
+    if (a.unit) {
+      float ss = 0.f;
+      if (VEC)
+        for (int e = 4 * lane; e < a.dk; e += 128) {
+          const float4 v = *reinterpret_cast<const float4*>(src + e);
+          ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+        }
+      else
+        for (int e = lane; e < a.dk; e += 32) ss = fmaf(src[e], src[e], ss);
+      sc = 1.0f / sqrtf(warp_sum(ss) / (float)a.dk + a.eps);
+    }
+    if (is_q && a.temp_every > 0) sc *= 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+    if (VEC)
+      for (int e = 4 * lane; e < a.dk; e += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(src + e);
+        store4(dst + e, make_float4(v.x * sc, v.y * sc, v.z * sc, v.w * sc));
+      }
+    else
+      for (int e = lane; e < a.dk; e += 32) dst[e] = from_f32<T>(src[e] * sc);
+    return;
+  }
+  if (seq < 0) return;
+  const int vh = hd - a.n_q - a.n_k;
+  const float* src = row + (size_t)(a.n_q + a.n_k) * a.dk + (size_t)vh * a.dv;
+  float* first = a.v_mode ? a.v_first + ((size_t)t * a.n_v + vh) * a.dv : nullptr;
+  T* dst = a.write_kv ? v_cache + kv_row_offset(a.vp, seq, a.tok_pos[t], vh) : nullptr;
+  const float keep = 1.0f - a.lambda;
+  if (VEC) {
+    for (int e = 4 * lane; e < a.dv; e += 128) {
+      float4 v = *reinterpret_cast<const float4*>(src + e);
+      if (a.v_mode == 1) *reinterpret_cast<float4*>(first + e) = v;
+      if (a.v_mode == 2) {
+        const float4 f = *reinterpret_cast<const float4*>(first + e);
+        v = make_float4(fmaf(keep, v.x, a.lambda * f.x), fmaf(keep, v.y, a.lambda * f.y), fmaf(keep, v.z, a.lambda * f.z),
+                        fmaf(keep, v.w, a.lambda * f.w));
+      }
+      if (dst) store4(dst + e, v);
+    }
+  } else {
+    for (int e = lane; e < a.dv; e += 32) {
+      float v = src[e];
+      if (a.v_mode == 1) first[e] = v;
+      if (a.v_mode == 2) v = fmaf(keep, v, a.lambda * first[e]);
+      if (dst) dst[e] = from_f32<T>(v);
+    }
+  }
+}
+
+template <typename T>
+static int launch_unit_prepare(const UnitPrepareArgs& a, void* k_cache, void* v_cache, void* q_out, bool vec, cudaStream_t stream) {
+  const long blocks = ((long)a.n_tokens * (a.n_q + a.n_k + a.n_v) + UP_WARPS - 1) / UP_WARPS;
+  if (blocks > 0x7fffffffL) return LLMI_ERR_BAD_SIZE;
+  if (vec)
+    return launch_pdl(PDL_ROPE, qkv_unit_prepare_kernel<T, true>, dim3((unsigned)blocks), dim3(UP_WARPS * 32), 0, stream, a, (T*)k_cache,
+                      (T*)v_cache, (T*)q_out);
+  return launch_pdl(PDL_ROPE, qkv_unit_prepare_kernel<T, false>, dim3((unsigned)blocks), dim3(UP_WARPS * 32), 0, stream, a, (T*)k_cache,
+                    (T*)v_cache, (T*)q_out);
+}
+
 template <typename T>
 static int launch_prepare_heads(const float* proj, long ld, int n_q_heads, int n_k_heads, int dk, int n_v_heads, int dv,
                                 const float* inv_freq, int rot_dims, int pairing, float amplitude, int v_from_k,
@@ -283,5 +402,27 @@ LLMI_EXPORT int llmi_qkv_prepare(int dtype, const float* proj, long ld, int n_q_
     return launch_pdl(PDL_SMALL, qkv_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(128), 0, stream, proj, ld, n_q_heads,
                       n_k_heads, dk, n_v_heads, dv, q_norm_w, k_norm_w, eps, inv_freq, rot_dims, pairing, amplitude, v_from_k, tok_seq, tok_pos, kp, vp,
                       (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, (__nv_bfloat16*)q_out, ldq, has_kv, write_kv);
+  return LLMI_ERR_BAD_DTYPE;
+}
+
+// See the head of this file.  v_first: fp32 [n_tokens, n_v_heads * dv] contiguous (v_mode 1: written, 2: read; 0: unused).
+LLMI_EXPORT int llmi_qkv_unit_prepare(int dtype, const float* proj, long ld, int n_q_heads, int n_k_heads, int dk, int n_v_heads,
+                                      int dv, int unit, float eps, float temp_coef, int temp_every, int v_mode, float lambda,
+                                      float* v_first, const int32_t* tok_seq, const int32_t* tok_pos, const int32_t* seq_pages,
+                                      int pages_stride, int page_size, void* k_cache, void* v_cache, void* q_out, long ldq,
+                                      int n_tokens, int write_kv, cudaStream_t stream) {
+  if (n_tokens <= 0 || n_q_heads <= 0 || n_k_heads <= 0 || n_v_heads <= 0 || dk <= 0 || dv <= 0 || page_size <= 0) return LLMI_ERR_BAD_SIZE;
+  if (temp_every < 0 || v_mode < 0 || v_mode > 2 || (v_mode && !v_first)) return LLMI_ERR_BAD_SIZE;
+  UnitPrepareArgs a;
+  a.proj = proj; a.ld = ld; a.n_q = n_q_heads; a.n_k = n_k_heads; a.dk = dk; a.n_v = n_v_heads; a.dv = dv;
+  a.unit = unit; a.eps = eps; a.temp_coef = temp_coef; a.temp_every = temp_every;
+  a.v_mode = v_mode; a.lambda = lambda; a.v_first = v_first; a.tok_seq = tok_seq; a.tok_pos = tok_pos;
+  a.kp = PagedKV{seq_pages, pages_stride, page_size, n_k_heads, dk};
+  a.vp = PagedKV{seq_pages, pages_stride, page_size, n_v_heads, dv};
+  a.ldq = ldq; a.n_tokens = n_tokens; a.write_kv = write_kv;
+  const bool vec = !(dk % 4) && !(dv % 4) && !(ld % 4) && !(ldq % 4) && !((uintptr_t)proj & 15) && !((uintptr_t)q_out & 15) &&
+                   !((uintptr_t)k_cache & 15) && !((uintptr_t)v_cache & 15) && !((uintptr_t)v_first & 15);
+  if (dtype == LLMI_DTYPE_F32) return launch_unit_prepare<float>(a, k_cache, v_cache, q_out, vec, stream);
+  if (dtype == LLMI_DTYPE_BF16) return launch_unit_prepare<__nv_bfloat16>(a, k_cache, v_cache, q_out, vec, stream);
   return LLMI_ERR_BAD_DTYPE;
 }

@@ -163,7 +163,8 @@ def lib():
                      "llmi_gdelta_prepare", "llmi_dplr_recurrence", "llmi_activate", "llmi_attention_maps_mma", "llmi_attention_maps_mma_supported", "llmi_tanh_rows", "llmi_norm_conv_token",
                      "llmi_layernorm", "llmi_depth_mix", "llmi_gate_rows", "llmi_pool_rows", "llmi_mix_layernorm",
                      "llmi_moe_identity_add", "llmi_channel_decay", "llmi_rows_activate", "llmi_decay_recurrence",
-                     "llmi_normed_pair", "llmi_stream_axpy_norm"):
+                     "llmi_normed_pair", "llmi_stream_axpy_norm", "llmi_stream_postnorm", "llmi_softcap_rows", "llmi_moe_table",
+                     "llmi_qkv_unit_prepare", "llmi_latent_prepare_direct"):
             getattr(l, name).restype = c_int
         l.llmi_gemm_tc_workspace.restype = c_long
         l.llmi_delta_state_floats.restype = c_long
@@ -177,7 +178,7 @@ def lib():
         l.llmi_gemm_tc.argtypes = [P, L, P, L, P, P, L, I, I, I, I, P, L, P, I, P, P]
         l.llmi_rmsnorm.argtypes = [I, P, P, P, P, I, I, F, P]
         l.llmi_rope_store.argtypes = [I, P, L, P, I, P, P, P, I, I, P, P, I, I, I, I, I, P]
-        l.llmi_attention_prefill_tc.argtypes = [P, L, L, P, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, I, P, L, P, I, P, I, P, P, L, P, I, P, L, P]
+        l.llmi_attention_prefill_tc.argtypes = [P, L, L, P, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, I, P, L, P, I, P, I, P, P, L, P, I, P, L, P, P, P, P]
         _configured = True
     return l
 
@@ -782,11 +783,12 @@ def prefill_split_jobs(q_lens, kv_lens, window: int, split_pages: int, pool: int
 
 def attention_prefill_tc(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, seq_pages, seq_q_start, seq_kv_len,
                          n_blocks: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0,
-                         split=None, pooled=None, gate=None) -> None:
+                         split=None, pooled=None, gate=None, bias=None, sink=None) -> None:
     """The same prompt attention on the tcgen05 tensor cores (head size 64 or 128); arguments as ``attention_prefill``.
     ``pooled = (pool, k_pool, v_pool, pool_pages)``: beside its window a query sees one pooled row per block of ``pool``
     positions that lies wholly before the window (row b of the sequence's pooled pages is block b; caches shaped as the
     token caches).  ``gate``: fp32 [tokens, >= n_heads]; head h's output is multiplied by logistic(gate[t, h]).
+    ``bias = (r1, r2)`` (not with ``pooled``) and ``sink``: see :func:`attention_flex`.
     ``split = (n_jobs, split_pages, workspace)``: cut the key range of every query block into jobs of
     ``split_pages`` pages (``n_jobs`` from :func:`prefill_split_jobs`, ``workspace`` fp32 of
     n_jobs * n_heads * (head_dim + 2) * 128 floats)."""
@@ -807,13 +809,14 @@ def attention_prefill_tc(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, s
     if gate is not None:
         _need_cuda(gate)
         assert gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == q.shape[0] and gate.shape[1] >= n_heads
+    r1, r2 = _bias_and_sink(bias, sink, n_heads)
     _check("attention_prefill_tc", lib().llmi_attention_prefill_tc(
         q.data_ptr(), q.stride(0), q.shape[0], out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
         k_cache.shape[0], seq_pages.data_ptr(), seq_pages.stride(0), seq_q_start.data_ptr(), seq_kv_len.data_ptr(), S,
         n_blocks, n_heads, n_kv_heads, head_dim, scale, window, n_jobs, split_pages, _addr(ws),
         ws.numel() if ws is not None else 0, sc.attn_tickets.data_ptr(), sc.N_ATTN_TICKETS, sc.error.data_ptr(), pool,
         _addr(k_pool), _addr(v_pool), k_pool.shape[0] if pool else 0, _addr(pool_pages), pool_pages.stride(0) if pool else 0,
-        _addr(gate), gate.stride(0) if gate is not None else 0, _stream_int()))
+        _addr(gate), gate.stride(0) if gate is not None else 0, _addr(r1), _addr(r2), _addr(sink), _stream_int()))
 
 
 # Which prompt-attention kernel runs: "tc" (tcgen05: about 43 us for a 2,048-token prompt of 32 heads of 64) or
@@ -944,9 +947,37 @@ def qkv_prepare(proj: torch.Tensor, n_q_heads: int, n_k_heads: int, dk: int, n_v
         _ptr(q_out), c_long(q_out.stride(0)), c_int(T), c_int(1 if has_kv else 0), c_int(1 if write_kv else 0), _stream()))
 
 
+VALUES_PLAIN, VALUES_KEEP, VALUES_MIX = 0, 1, 2
+
+
+def qkv_unit_prepare(proj: torch.Tensor, n_q_heads: int, n_k_heads: int, dk: int, n_v_heads: int, dv: int, ctx, seq_pages,
+                     page_size: int, k_cache, v_cache, q_out: torch.Tensor, unit_eps: float | None = None, temperature=None,
+                     value_mode: int = VALUES_PLAIN, lam: float = 0.0, v_first: torch.Tensor | None = None,
+                     write_kv: bool = True) -> None:
+    """From the fp32 rows [q | k | v] of a step, without a rotation: q into ``q_out`` (compute type), k and v into their
+    cache pages.  ``unit_eps``: every q and k head is divided by sqrt(mean(x^2) + unit_eps).  ``temperature`` = (coef,
+    every): q at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).  ``value_mode``: VALUES_KEEP also
+    writes the values to ``v_first`` (fp32 [T, n_v_heads * dv]), VALUES_MIX makes them (1 - lam) v + lam v_first."""
+    _need_cuda(proj, seq_pages, k_cache, v_cache, q_out, v_first)
+    T = proj.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= n_q_heads * dk + n_k_heads * dk + n_v_heads * dv
+    assert q_out.shape == (T, n_q_heads * dk) and q_out.stride(1) == 1 and seq_pages.dtype == torch.int32
+    assert k_cache.dtype == v_cache.dtype == q_out.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[-3:] == (n_k_heads, page_size, dk) and v_cache.shape[-3:] == (n_v_heads, page_size, dv)
+    if value_mode != VALUES_PLAIN:
+        assert v_first is not None and v_first.dtype == torch.float32 and v_first.is_contiguous() and v_first.shape == (T, n_v_heads * dv)
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    _check("qkv_unit_prepare", lib().llmi_qkv_unit_prepare(
+        c_int(_dtype_code(q_out)), _ptr(proj), c_long(proj.stride(0)), c_int(n_q_heads), c_int(n_k_heads), c_int(dk), c_int(n_v_heads),
+        c_int(dv), c_int(0 if unit_eps is None else 1), c_float(unit_eps or 0.0), c_float(coef), c_int(every), c_int(value_mode),
+        c_float(lam), _ptr(v_first), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(seq_pages), c_int(seq_pages.stride(0)),
+        c_int(page_size), _ptr(k_cache), _ptr(v_cache), _ptr(q_out), c_long(q_out.stride(0)), c_int(T), c_int(1 if write_kv else 0),
+        _stream()))
+
+
 def attention_flex(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, ctx, seq_pages, page_size: int, n_heads: int,
                    n_kv_heads: int, maps: int, dk: int, dv: int, scale: float, head_scale=None, window: int = 0,
-                   chunk: int = 0, pooled=None, gate=None, softcap: float = 0.0) -> None:
+                   chunk: int = 0, pooled=None, gate=None, softcap: float = 0.0, bias=None, sink=None) -> None:
     """Causal attention of every token over its sequence's cache with ``maps`` score maps per head (query row
     [head][map][dk], key heads [kv head][map], one set of values [kv head][dv]); out [T, heads*maps*dv] in q's type or
     fp32.  ``head_scale`` fp32 [heads] multiplies the scores of a head; ``window`` and ``chunk`` limit the visible keys
@@ -954,7 +985,10 @@ def attention_flex(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, ctx, se
     beside its window a query sees row b of the pooled pages for every block b of ``pool`` positions that lies wholly
     before the window (b * pool + pool - 1 <= p - window), in the same softmax.  ``gate`` fp32 [T, >= heads] (row-strided):
     head h's output is multiplied by logistic(gate[t, h]); a gate of exactly heads*dv columns (one map) has a number per
-    output entry instead.  ``softcap`` > 0: a score s becomes softcap * tanh(s / softcap) before the softmax."""
+    output entry instead.  ``softcap`` > 0: a score s becomes softcap * tanh(s / softcap) before the softmax.  ``bias`` =
+    (r1, r2), fp32 [heads] each (not with ``pooled``): a key d positions back then loses r1 * ln(1 + r2 * d) of its score.
+    ``sink`` fp32 [heads]: exp(sink) joins the head's softmax sum and stands for no key."""
+    r1, r2 = _bias_and_sink(bias, sink, n_heads)
     gate_per = _gate_per(gate, n_heads, maps, dv)
     _need_cuda(q, out, k_cache, v_cache, seq_pages, head_scale, gate)
     T = q.shape[0]
@@ -975,7 +1009,15 @@ def attention_flex(q: torch.Tensor, out: torch.Tensor, k_cache, v_cache, ctx, se
         _ptr(seq_pages), c_int(seq_pages.stride(0)), c_int(page_size), c_int(T), c_int(n_heads), c_int(n_kv_heads), c_int(maps),
         c_int(dk), c_int(dv), c_float(scale), _ptr(head_scale), c_int(window), c_int(chunk), c_int(pool), _ptr(k_pool), _ptr(v_pool),
         _ptr(pool_pages), c_int(pool_pages.stride(0) if pool else 0), _ptr(gate), c_long(gate.stride(0) if gate is not None else 0),
-        c_int(gate_per), c_float(softcap), _stream()))
+        c_int(gate_per), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink), _stream()))
+
+
+def _bias_and_sink(bias, sink, n_heads: int) -> tuple:
+    """The two tensors of a bias by distance (or None, None); both, and a sink, are one fp32 number per head."""
+    r1, r2 = bias if bias is not None else (None, None)
+    for t in (r1, r2, sink):
+        assert t is None or (t.is_cuda and t.dtype == torch.float32 and t.numel() == n_heads and t.is_contiguous())
+    return r1, r2
 
 
 def _gate_per(gate, n_heads: int, maps: int, dv: int) -> int:
@@ -1004,7 +1046,7 @@ def pool_rows(k_cache, v_cache, seq_pages, k_pool, v_pool, pool_pages, page_size
 
 def attention_maps(q, out, k_cache, v_cache, ctx, seq_pages, page_size: int, n_heads: int, n_kv_heads: int, maps: int,
                    dk: int, dv: int, scale: float, head_scale=None, window: int = 0, chunk: int = 0, rt=None, pooled=None,
-                   gate=None, softcap: float = 0.0) -> None:
+                   gate=None, softcap: float = 0.0, bias=None, sink=None) -> None:
     """The attention of a step in its general form (arguments as :func:`attention_flex`): bf16 sizes that the
     tensor-core kernel takes go there — prompts as blocks of 128 query rows, steps of single tokens cut over the
     positions (``rt`` lends the workspace of the cuts) —, everything else, and the 32-bit path, to the generic kernel."""
@@ -1028,7 +1070,7 @@ def attention_maps(q, out, k_cache, v_cache, ctx, seq_pages, page_size: int, n_h
                 ws = rt.scratch("attn_prefill_partials", (jobs * n_heads * (dk + 2) * 128,), torch.float32)
                 split = (jobs, PREFILL_SPLIT_PAGES, ws)
         attention_prefill_tc(q, out, k_cache, v_cache, seq_pages, ctx.seq_q_start, ctx.seq_kv_len, n_q_blocks, n_heads,
-                             n_kv_heads, dk, scale, window, split, pooled if pool else None, gate)
+                             n_kv_heads, dk, scale, window, split, pooled if pool else None, gate, bias, sink)
         return
     if (q.dtype == torch.bfloat16 and rt is not None and _MAPS_ATTENTION == "mma" and not _FORCE_GENERIC_ATTENTION
             and lib().llmi_attention_maps_mma_supported(c_int(dk), c_int(dv), c_int(n_heads // n_kv_heads), c_int(page_size))
@@ -1046,6 +1088,7 @@ def attention_maps(q, out, k_cache, v_cache, ctx, seq_pages, page_size: int, n_h
         assert q.stride(1) == 1 and out.stride(1) == 1 and out.shape == (T, n_heads * maps * dv) and k_cache.is_contiguous()
         assert v_cache.is_contiguous() and k_cache.shape[-3:] == (n_kv_heads * maps, page_size, dk)
         assert v_cache.shape[-3:] == (n_kv_heads, page_size, dv) and out.dtype in (torch.bfloat16, torch.float32)
+        r1, r2 = _bias_and_sink(bias, sink, n_heads)
         prompt = not ctx.decode
         splits, pps, ws, n_ws = 1, max(P, 1), None, 0
         if not prompt:
@@ -1059,10 +1102,11 @@ def attention_maps(q, out, k_cache, v_cache, ctx, seq_pages, page_size: int, n_h
             c_int(dv), c_float(scale), _ptr(head_scale), c_int(window), c_int(chunk), c_int(1 if prompt else 0),
             c_int(T // 128 + S), c_int(splits), c_int(pps), _ptr(ws), c_long(n_ws), c_int(pool), _ptr(k_pool), _ptr(v_pool),
             _ptr(pool_pages), c_int(pool_pages.stride(0) if pool else 0), _ptr(gate),
-            c_long(gate.stride(0) if gate is not None else 0), c_int(gate_per), c_float(softcap), _stream()))
+            c_long(gate.stride(0) if gate is not None else 0), c_int(gate_per), c_float(softcap), _ptr(r1), _ptr(r2), _ptr(sink),
+            _stream()))
         return
     attention_flex(q, out, k_cache, v_cache, ctx, seq_pages, page_size, n_heads, n_kv_heads, maps, dk, dv, scale, head_scale,
-                   window, chunk, pooled, gate, softcap)
+                   window, chunk, pooled, gate, softcap, bias, sink)
 
 
 _MAPS_ATTENTION = os.environ.get("LLMI_MAPS_ATTENTION", "mma")      # "generic": the fp32-arithmetic kernel for everything
@@ -1235,9 +1279,10 @@ def linear_batched(x: torch.Tensor, bx: int, w: torch.Tensor, out: torch.Tensor,
 # Latent attention
 
 def latent_prepare(down: torch.Tensor, Q: int, C: int, R: int, wq, wc, eps: float, inv_freq, rot_dims: int, ctx, seq_pages,
-                   page_size: int, cache: torch.Tensor, cq: torch.Tensor, write_kv: bool = True) -> None:
+                   page_size: int, cache: torch.Tensor, cq: torch.Tensor, write_kv: bool = True, pairing: int = 1) -> None:
     """From the fp32 down-projection rows [query latent Q | latent C | shared key part R]: the RMS-normed query
-    latent into ``cq`` (compute type) and the cache row [normed latent | rotated key part] of every token."""
+    latent into ``cq`` (compute type) and the cache row [normed latent | rotated key part] of every token.  ``pairing``:
+    which entries turn together, 1 neighbours (2i, 2i + 1), 0 entries (i, i + rot_dims/2)."""
     _need_cuda(down, wq, wc, inv_freq, seq_pages, cache, cq)
     T = down.shape[0]
     assert down.dtype == torch.float32 and down.stride(1) == 1 and down.shape[1] >= Q + C + R
@@ -1246,10 +1291,30 @@ def latent_prepare(down: torch.Tensor, Q: int, C: int, R: int, wq, wc, eps: floa
     _check("latent_prepare", lib().llmi_latent_prepare(
         c_int(_dtype_code(cq)), _ptr(down), c_long(down.stride(0)), c_int(Q), c_int(C), c_int(R), _ptr(wq), _ptr(wc), c_float(eps),
         _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(seq_pages), c_int(seq_pages.stride(0)),
-        c_int(page_size), _ptr(cache), _ptr(cq), c_int(T), c_int(1 if write_kv else 0), _stream()))
+        c_int(page_size), _ptr(cache), _ptr(cq), c_int(T), c_int(1 if write_kv else 0), c_int(pairing), _stream()))
 
 
-def latent_q_rotate(q: torch.Tensor, D: int, qa: torch.Tensor, C: int, R: int, H: int, inv_freq, rot_dims: int, ctx) -> None:
+def latent_prepare_direct(proj: torch.Tensor, H: int, D: int, C: int, R: int, wc, eps: float, inv_freq, rot_dims: int, pairing: int, ctx,
+                          seq_pages, page_size: int, cache: torch.Tensor, qn: torch.Tensor, qa: torch.Tensor,
+                          write_kv: bool = True) -> None:
+    """The same for queries that come straight from the layer's input: from the fp32 rows [q: H*(D+R) | latent C | shared
+    key part R], the plain part of every head's query into ``qn`` [T, H*D], its rotated part behind the C leading entries
+    of the head's row of ``qa`` [T, H*(C+R)], and the cache row of every token."""
+    _need_cuda(proj, wc, inv_freq, seq_pages, cache, qn, qa)
+    T = proj.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= H * (D + R) + C + R
+    assert qn.shape == (T, H * D) and qn.is_contiguous() and qa.shape == (T, H * (C + R)) and qa.stride(1) == 1
+    assert qn.dtype == qa.dtype == cache.dtype and cache.is_contiguous() and cache.shape[-1] == C + R and cache.shape[-3] == 1
+    assert cache.shape[-2] == page_size and wc.dtype == torch.float32 and wc.numel() == C and inv_freq.numel() >= rot_dims // 2
+    _check("latent_prepare_direct", lib().llmi_latent_prepare_direct(
+        c_int(_dtype_code(qn)), _ptr(proj), c_long(proj.stride(0)), c_int(H), c_int(D), c_int(C), c_int(R), _ptr(wc), c_float(eps),
+        _ptr(inv_freq), c_int(rot_dims), c_int(pairing), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(seq_pages),
+        c_int(seq_pages.stride(0)), c_int(page_size), _ptr(cache), _ptr(qn), _ptr(qa), c_long(qa.stride(0)), c_int(T),
+        c_int(1 if write_kv else 0), _stream()))
+
+
+def latent_q_rotate(q: torch.Tensor, D: int, qa: torch.Tensor, C: int, R: int, H: int, inv_freq, rot_dims: int, ctx,
+                    pairing: int = 1) -> None:
     """The part of every head's query that is rotated by position, q[:, h, D:], into qa[:, h, C:]."""
     _need_cuda(q, qa, inv_freq)
     T = q.shape[0]
@@ -1257,7 +1322,7 @@ def latent_q_rotate(q: torch.Tensor, D: int, qa: torch.Tensor, C: int, R: int, H
     assert q.shape[1] == H * (D + R) and qa.shape == (T, H * (C + R))
     _check("latent_q_rotate", lib().llmi_latent_q_rotate(
         c_int(_dtype_code(q)), _ptr(q), c_long(q.stride(0)), c_int(D), _ptr(qa), c_long(qa.stride(0)), c_int(C), c_int(R), c_int(H),
-        _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), c_int(T), _stream()))
+        _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), c_int(T), c_int(pairing), _stream()))
 
 
 _LATENT_ATTENTION = os.environ.get("LLMI_LATENT_ATTENTION", "mma")      # "generic": the fp32-arithmetic kernel for everything
@@ -1266,7 +1331,7 @@ _LATENT_ATTENTION = os.environ.get("LLMI_LATENT_ATTENTION", "mma")      # "gener
 _LATENT_BLOCKS_PER_SM = int(os.environ.get("LLMI_LATENT_BLOCKS_PER_SM", "2"))
 
 
-def latent_attention_plan(ctx, n_tokens: int, n_pages: int, H: int) -> tuple:
+def latent_attention_plan(ctx, n_tokens: int, n_pages: int, H: int, window: int = 0, page_size: int = 64) -> tuple:
     """(cuts over the positions, pages per cut) of the tensor-core latent attention for a step: prompts are not cut;
     a step of single tokens is cut until about two blocks per SM are at work (the kernel keeps one page buffer
     then, so two blocks share an SM; measured, batch 8 at 4,096 positions: 0.853 ms a step with one block per SM, 0.831
@@ -1274,6 +1339,8 @@ def latent_attention_plan(ctx, n_tokens: int, n_pages: int, H: int) -> tuple:
     only, so a recorded step can be replayed."""
     if not ctx.decode:
         return 1, max(n_pages, 1)
+    if window > 0:      # a query sees at most the pages its window spans
+        n_pages = min(n_pages, -(-window // page_size) + 1)
     hpb = 1
     while hpb < H and hpb < 16:
         hpb *= 2
@@ -1284,8 +1351,8 @@ def latent_attention_plan(ctx, n_tokens: int, n_pages: int, H: int) -> tuple:
 
 
 def attention_latent(qa: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, ctx, seq_pages, page_size: int, H: int, C: int,
-                     R: int, scale: float, rt=None) -> None:
-    """Causal attention of every token's heads over its sequence's latent rows: scores from all C + R entries of a
+                     R: int, scale: float, rt=None, window: int = 0) -> None:
+    """Causal attention of every token's heads over its sequence's latent rows (``window`` > 0: the last ``window`` of them): scores from all C + R entries of a
     row, context from its first C.  qa [T, H*(C+R)], out [T, H*C].  bf16 sizes that the tensor-core kernel takes go
     there (``rt`` lends the workspace of its cuts); everything else, and the 32-bit path, to the generic kernel."""
     _need_cuda(qa, out, cache, seq_pages)
@@ -1295,18 +1362,18 @@ def attention_latent(qa: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, c
     if (qa.dtype == torch.bfloat16 and rt is not None and _LATENT_ATTENTION == "mma"
             and lib().llmi_attention_latent_mma_supported(c_int(C), c_int(R), c_int(page_size))
             and qa.data_ptr() % 16 == 0 and qa.stride(0) % 8 == 0):
-        splits, pps = latent_attention_plan(ctx, T, seq_pages.shape[1], H)
+        splits, pps = latent_attention_plan(ctx, T, seq_pages.shape[1], H, window, page_size)
         n_ws = int(lib().llmi_attention_latent_mma_workspace(c_int(T), c_int(H), c_int(C), c_int(splits)))
         ws = rt.scratch("latent_partials", (n_ws,), torch.float32) if n_ws else None
         _check("attention_latent_mma", lib().llmi_attention_latent_mma(
             _ptr(qa), c_long(qa.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(cache), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos),
             _ptr(seq_pages), c_int(seq_pages.stride(0)), c_int(page_size), c_int(T), c_int(H), c_int(C), c_int(R), c_float(scale),
-            c_int(splits), c_int(pps), c_int(1 if ctx.decode else 2), _ptr(ws), c_long(n_ws), _stream()))
+            c_int(splits), c_int(pps), c_int(1 if ctx.decode else 2), _ptr(ws), c_long(n_ws), c_int(window), _stream()))
         return
     _check("attention_latent", lib().llmi_attention_latent(
         c_int(_dtype_code(qa)), _ptr(qa), c_long(qa.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(cache), _ptr(ctx.tok_seq),
         _ptr(ctx.tok_pos), _ptr(seq_pages), c_int(seq_pages.stride(0)), c_int(page_size), c_int(T), c_int(H), c_int(C), c_int(R),
-        c_float(scale), _stream()))
+        c_float(scale), c_int(window), _stream()))
 
 
 # ---------------------------------------------------------------------------------------------
@@ -1440,6 +1507,18 @@ def moe_route(logits: torch.Tensor, top: int, ctx, idx: torch.Tensor, wt: torch.
     _check("moe_route", lib().llmi_moe_route(_ptr(logits), c_long(logits.stride(0)), c_int(E), c_int(top), c_int(mode),
                                              c_int(n_groups), c_int(keep), _ptr(ctx.tok_seq), _ptr(idx), _ptr(wt), c_int(T),
                                              _ptr(correction), c_float(scale), c_int(identity), _ptr(id_wt), _stream()))
+
+
+def moe_table(table: torch.Tensor, token_ids: torch.Tensor, ctx, idx: torch.Tensor, wt: torch.Tensor) -> None:
+    """No router: idx int32 [T, top] = table[token_ids[t]] (table int32 [vocab, top]) and wt fp32 [T, top] = 1 / top; a token
+    row of no sequence gets index -1."""
+    _need_cuda(table, token_ids, idx, wt)
+    V, top = table.shape
+    T = token_ids.shape[0]
+    assert table.dtype == token_ids.dtype == idx.dtype == torch.int32 and table.is_contiguous() and wt.dtype == torch.float32
+    assert idx.shape == (T, top) and wt.shape == (T, top) and idx.is_contiguous() and wt.is_contiguous()
+    _check("moe_table", lib().llmi_moe_table(_ptr(table), c_int(V), c_int(top), _ptr(token_ids), _ptr(ctx.tok_seq), _ptr(idx), _ptr(wt),
+                                             c_int(T), _stream()))
 
 
 def moe_identity_add(h: torch.Tensor, id_wt: torch.Tensor, y: torch.Tensor) -> None:
@@ -1580,3 +1659,24 @@ def stream_axpy_norm(x: torch.Tensor, y: torch.Tensor, m: float, norm_w: torch.T
         assert norm_w.dtype == torch.float32 and norm_w.numel() == W and h.shape == (T, W) and h.is_contiguous()
     _check("stream_axpy_norm", lib().llmi_stream_axpy_norm(_ptr(x), _ptr(y), c_float(m), c_int(T), c_int(W), _ptr(norm_w), c_float(eps),
                                                            c_int(_dtype_code(h) if h is not None else 0), _ptr(h), _stream()))
+
+
+def stream_postnorm(x: torch.Tensor, y: torch.Tensor | None, alpha: float, norm_w: torch.Tensor | None, eps: float,
+                    h: torch.Tensor | None = None) -> None:
+    """x = norm_w * v / rms(v) with v = alpha * x + y (fp32 [T, W], contiguous), and ``h`` [T, W] (compute type, contiguous,
+    optional) = the new x.  Without ``y`` and ``norm_w``: only h = x."""
+    _need_cuda(x, y, norm_w, h)
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and (y is None) == (norm_w is None)
+    assert y is None or (y.dtype == torch.float32 and y.is_contiguous() and y.shape == (T, W) and norm_w.dtype == torch.float32
+                         and norm_w.numel() == W)
+    assert h is None or (h.shape == (T, W) and h.is_contiguous())
+    _check("stream_postnorm", lib().llmi_stream_postnorm(_ptr(x), _ptr(y), c_float(alpha), c_int(T), c_int(W), _ptr(norm_w), c_float(eps),
+                                                         c_int(_dtype_code(h) if h is not None else 0), _ptr(h), _stream()))
+
+
+def softcap_rows(v: torch.Tensor, cap: float) -> None:
+    """v = cap * tanh(v / cap) in place; fp32, contiguous."""
+    _need_cuda(v)
+    assert v.dtype == torch.float32 and v.is_contiguous() and cap > 0
+    _check("softcap_rows", lib().llmi_softcap_rows(_ptr(v), c_long(v.numel()), c_float(cap), _stream()))

@@ -461,3 +461,80 @@ class GatedAttention(_MapsAttention):
                                softcap=self.softcap)
         kernels.linear(out, self.w_o, x, self.b_o, kernels.OUT_STORE_F32 if store else kernels.OUT_ADD_F32)
         return False
+
+
+@part("mixer", "distance_attention")
+class DistanceAttention(_MapsAttention):
+    """Softmax attention of grouped queries without a rotation; what positions do is a bias on the scores.  Optional pieces,
+    each a parameter:
+
+    * ``unit_qk``: every q and k head is divided by its root mean square over ``dim`` (eps inside the root, no weight);
+    * ``temperature`` = (coef, every): q at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1);
+    * ``distance_bias``: a key d positions back loses r1_h * ln(1 + r2_h * d) of its score, two learned numbers per head;
+    * ``sink``: exp(sink_h), one learned number per head, joins the softmax's sum and stands for no key;
+    * ``value_mix``: ``"first"`` — the layer's values are kept for the rest of the step; ``"later"`` — the values are
+      (1 - lambda) v + lambda v_first with the kept values of the same token and a learned lambda; the mixed values are
+      what the cache holds, so nothing of the first layer is needed for earlier tokens;
+    * ``window``: the last ``window`` positions only.
+
+    params: ``width``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale``, ``eps`` (of ``unit_qk``), and the above.
+    tensors: ``q`` [heads*dim, width], ``k`` [kv_heads*dim, width], ``v`` [kv_heads*vdim, width], ``o`` [width, heads*vdim];
+    with ``distance_bias`` ``r1``, ``r2`` [heads]; with ``sink`` ``sink`` [heads]; with ``value_mix`` ``"later"`` ``vmix``
+    (a scalar)."""
+    stores_output = True
+
+    @classmethod
+    def declare(cls, spec):
+        p = spec.params
+        d = cls._declare_projections(p, 1)
+        H = p["heads"]
+        if p.get("distance_bias", False):
+            d.update({"r1": TensorDecl((H,), "norm_scale"), "r2": TensorDecl((H,), "norm_scale")})
+        if p.get("sink", False):
+            d["sink"] = TensorDecl((H,), "bias")
+        if p.get("value_mix") == "later":
+            d["vmix"] = TensorDecl((), "bias")
+        return d
+
+    def __init__(self, spec, tensors, rt, **_):
+        p = dict(spec.params)
+        p.setdefault("eps", 0.0)
+        self.rt = rt
+        self._sizes(p)
+        if self.shares_kv or self.chunk:
+            raise ValueError("distance_attention: has key and value projections of its own and no mask of blocks")
+        self._projections(tensors, rt)
+        self.unit_eps = self.eps if p.get("unit_qk", False) else None
+        self.temperature = None
+        if p.get("temperature") is not None:
+            coef, every = p["temperature"]
+            if int(every) < 1:
+                raise ValueError("distance_attention: the temperature's step is at least one position")
+            self.temperature = (float(coef), int(every))
+        self.bias = self.sink = None
+        if p.get("distance_bias", False):
+            self.bias = (rt.to_f32(tensors["r1"]), rt.to_f32(tensors["r2"]))
+        if p.get("sink", False):
+            self.sink = rt.to_f32(tensors["sink"])
+        mix = p.get("value_mix")
+        if mix not in (None, "first", "later"):
+            raise ValueError(f"distance_attention: value_mix is 'first' or 'later', not {mix!r}")
+        self.value_mode = {None: kernels.VALUES_PLAIN, "first": kernels.VALUES_KEEP, "later": kernels.VALUES_MIX}[mix]
+        self.lam = float(tensors["vmix"].float().item()) if mix == "later" else 0.0
+
+    def forward(self, h, x, ctx, binding, store: bool = False, then_norm=None) -> bool:
+        T = h.shape[0]
+        rt, H, G, D, Dv = self.rt, self.H, self.G, self.D, self.Dv
+        proj = rt.scratch("attn_proj", (T, self.w_in.shape[0]), torch.float32)
+        kernels.linear(h, self.w_in, proj, None, kernels.OUT_STORE_F32)
+        g = binding.group
+        pages = ctx.pages_of(g)
+        k_cache, v_cache = g.k[binding.index], g.v[binding.index]
+        q = rt.scratch("attn_q", (T, H * D))
+        first = rt.scratch("first_values", (T, G * Dv), torch.float32) if self.value_mode != kernels.VALUES_PLAIN else None
+        kernels.qkv_unit_prepare(proj, H, G, D, G, Dv, ctx, pages, g.page_size, k_cache, v_cache, q, self.unit_eps, self.temperature,
+                                 self.value_mode, self.lam, first, write_kv=binding.writes)
+        out = rt.scratch("attn_out", (T, H * Dv))
+        kernels.attention_maps(q, out, k_cache, v_cache, ctx, pages, g.page_size, H, G, 1, D, Dv, self.scale, None, self.window, 0,
+                               rt=rt, bias=self.bias, sink=self.sink)
+        return self._project_out(out, x, store, then_norm)

@@ -143,6 +143,55 @@ class ScaledParallelBlock:
         return None
 
 
+class StreamCopy:
+    """What a block says its first branch reads (``entry_norm``) when that is the stream itself: a copy of it in the
+    compute type, which whoever changes the stream last may make in the same pass and hand in as ``entry``."""
+
+
+@part("block", "postnorm")
+class PostNormBlock:
+    """The norm stands BEHIND the sum and replaces the stream, and the branches read the stream itself:
+    x = n1(a x + mixer(x));  x = n2(a x + ffn(x)) with a constant a.  The feed-forward (with its norm) may be absent.  The
+    branches write into an fp32 buffer of their own (both must take ``store=``); the norm offers ``replace_sum(x, y, a, h)``,
+    which joins, normalises and leaves the copy that the next branch reads in one pass.
+
+    Slots: ``mixer``, ``mixer_norm``, optional ``ffn`` and ``ffn_norm``.  Parameter: ``alpha`` (a)."""
+
+    def __init__(self, mixer, mixer_norm, ffn=None, ffn_norm=None, alpha: float = 1.0):
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("postnorm: a feed-forward comes with its norm, or not at all")
+        for p in (mixer, ffn):
+            if p is not None and not getattr(p, "stores_output", False):
+                raise ValueError(f"postnorm: the part {getattr(p, 'kind', p)!r} cannot store its output (store=)")
+        for n in (mixer_norm, ffn_norm):
+            if n is not None and not hasattr(n, "replace_sum"):
+                raise ValueError(f"postnorm: the norm {getattr(n, 'kind', n)!r} cannot replace the sum it reads (replace_sum)")
+        self.mixer, self.mixer_norm, self.ffn, self.ffn_norm = mixer, mixer_norm, ffn, ffn_norm
+        self.alpha = float(alpha)
+        self.rt = mixer_norm.rt
+
+    @property
+    def takes_padding_rows(self) -> bool:
+        return True          # rows are treated alone
+
+    entry_norm = StreamCopy()
+
+    def forward(self, x, ctx, binding, entry=None, next_norm=None):
+        shape = tuple(x.shape)
+        exact = self.rt.dtype == torch.float32            # the stream is its own copy
+        h = None if exact else self.rt.scratch("stream_copy", shape)
+        if not exact and entry is None:
+            kernels.stream_postnorm(x, None, 1.0, None, 0.0, h)
+        y = self.rt.scratch("branch_out", shape, torch.float32)
+        self.mixer.forward(x if exact else h, y, ctx, binding, store=True)
+        goes_on = isinstance(next_norm, StreamCopy)
+        self.mixer_norm.replace_sum(x, y, self.alpha, h if (self.ffn is not None or goes_on) else None)
+        if self.ffn is not None:
+            self.ffn.forward(x if exact else h, y, ctx, store=True)
+            self.ffn_norm.replace_sum(x, y, self.alpha, h if goes_on else None)
+        return h if goes_on else None
+
+
 @part("block", "prepost")
 class PrePostNormBlock:
     """A norm ahead of AND behind each sublayer:  x += post1(mixer(pre1(x)));  x += post2(ffn(pre2(x))).

@@ -51,8 +51,8 @@ class TokenTable:
 
 @part("head", "linear_head")
 class LinearHead:
-    """params: ``vocab``, ``width``, ``tied``, optional ``tensor`` (the matrix's local name; default ``weight``).
-    tensors: the matrix [vocab, width] unless tied."""
+    """params: ``vocab``, ``width``, ``tied``, optional ``tensor`` (the matrix's local name; default ``weight``),
+    optional ``softcap`` (0: none; a logit z becomes softcap * tanh(z / softcap)).  tensors: the matrix [vocab, width] unless tied."""
     takes_padding_rows = True       # token rows of no sequence (a step padded to a shape) do no harm: rows are treated alone
 
     @classmethod
@@ -64,6 +64,7 @@ class LinearHead:
     def __init__(self, spec, tensors, rt, embedding=None, **_):
         self.rt = rt
         self.vocab, self.width = int(spec.params["vocab"]), int(spec.params["width"])
+        self.softcap = float(spec.params.get("softcap", 0.0) or 0.0)
         self.tied = bool(spec.params.get("tied", False))
         if self.tied:
             if embedding is None:
@@ -78,4 +79,6 @@ class LinearHead:
     def forward(self, h_rows):
         logits = self.rt.scratch("logits", (h_rows.shape[0], self.vocab), torch.float32)
         kernels.linear(h_rows, self.weight, logits, None, kernels.OUT_STORE_F32)
+        if self.softcap > 0.0:
+            kernels.softcap_rows(logits, self.softcap)
         return logits

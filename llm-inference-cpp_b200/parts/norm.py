@@ -12,17 +12,21 @@ from .registry import TensorDecl, part
 class RMSNorm:
     """params: ``width``, ``eps``, optional ``tensor`` (the weight's local name; default ``weight``), optional
     ``one_plus`` (the file stores the weight around zero: y = (1 + w) · x · rsqrt(mean(x²) + eps); the sum 1 + w is made
-    once at load, in fp32).  tensors: the weight [width] (kept in fp32)."""
+    once at load, in fp32), optional ``one_gain`` (the file stores ONE number, which every coordinate is multiplied by).
+    tensors: the weight [width] (kept in fp32), or a scalar with ``one_gain``."""
     takes_padding_rows = True       # token rows of no sequence (a step padded to a shape) do no harm: rows are treated alone
 
     @classmethod
     def declare(cls, spec):
-        return {spec.params.get("tensor", "weight"): TensorDecl((spec.params["width"],), "norm_scale")}
+        shape = () if spec.params.get("one_gain", False) else (spec.params["width"],)
+        return {spec.params.get("tensor", "weight"): TensorDecl(shape, "norm_scale")}
 
     def __init__(self, spec, tensors, rt, **_):
         self.width = int(spec.params["width"])
         self.eps = float(spec.params["eps"])
         self.weight = rt.to_f32(tensors[spec.params.get("tensor", "weight")])
+        if spec.params.get("one_gain", False):       # one number for all: a row of it, so that every kernel reads a weight per entry
+            self.weight = self.weight.expand(self.width).contiguous()
         if spec.params.get("one_plus", False):
             self.weight = (self.weight + 1.0).contiguous()
         self.rt = rt
@@ -39,6 +43,10 @@ class RMSNorm:
         out = self.rt.scratch(scratch_name, (x.shape[0], self.width))
         kernels.stream_axpy_norm(x, y, m, self.weight, self.eps, out)
         return out
+
+    def replace_sum(self, x, y, alpha: float, h=None) -> None:
+        """x = this norm of (alpha * x + y), in one pass over the rows; ``h`` (compute type, optional) receives the new x."""
+        kernels.stream_postnorm(x, y, alpha, self.weight, self.eps, h)
 
     def deferred(self, n_tokens: int, name: str):
         """This norm for ``n_tokens`` rows as a :class:`kernels.DeferredNorm` — to be filled by the product

@@ -82,6 +82,7 @@ class TensorDecl:
     # "matrix" | "norm_scale" | "bias" | "table" | "mix": floating tensors (the role says how random weights draw them);
     # "int_table": the only role a file may store as integers
     role: str = "matrix"
+    high: int = 0                   # of an int_table: entries are 0 .. high - 1 (random weights: the entries of a row differ)
 
 
 def register_part(family: str, kind: str, cls: type, *, replace: bool = False) -> None:

@@ -3,7 +3,8 @@
 The reference builds random models only in its tests
 (tests/transformer_test.cpp:162-197: normal matrices, norm weights around one,
 written as an in-memory safetensors blob).  Here it is a mode of the library:
-matrices, tables and biases are N(0, 0.02), norm scales are 1 + N(0, 0.1), each
+matrices, tables and biases are N(0, 0.02), norm scales are 1 + N(0, 0.1),
+integer tables hold different numbers below their bound in every row; each
 tensor drawn from its own generator keyed by (seed, tensor name), so a tensor's
 values do not depend on which other tensors exist or in which order they are made.
 """
@@ -29,8 +30,14 @@ def _tensor_seed(seed: int, name: str) -> int:
     return int.from_bytes(digest[:8], "little") & ((1 << 63) - 1)
 
 
-def random_tensor(name: str, shape, role: str, seed: int, device="cpu") -> torch.Tensor:
-    """One fp32 tensor of the given role, reproducible from (seed, name) on a given device type."""
+def random_tensor(name: str, shape, role: str, seed: int, device="cpu", high: int = 0) -> torch.Tensor:
+    """One tensor of the given role (fp32; an ``int_table`` int32 with entries below ``high``), reproducible from (seed, name)
+    on a given device type."""
+    if role == "int_table" and len(shape) == 2 and 1 <= int(shape[1]) <= high:
+        gen = torch.Generator(device=device)
+        gen.manual_seed(_tensor_seed(seed, name))
+        order = torch.rand((int(shape[0]), high), generator=gen, device=device).argsort(dim=1)
+        return order[:, :int(shape[1])].to(torch.int32).contiguous()
     if role not in ("matrix", "norm_scale", "bias", "table", "mix"):
         raise ValueError(f"random weights: no rule for a tensor of role {role!r} ({name})")
     gen = torch.Generator(device=device)
@@ -45,8 +52,11 @@ def random_tensor(name: str, shape, role: str, seed: int, device="cpu") -> torch
 
 def random_tensors(spec, seed: int, device="cpu", dtype=torch.float32) -> dict:
     """All tensors a ModelSpec expects, drawn in fp32 and rounded once to ``dtype``."""
-    return {name: random_tensor(name, resolved_shape(d.shape), d.role, seed, device).to(dtype)
-            for name, d in expected_tensors(spec).items()}
+    out = {}
+    for name, d in expected_tensors(spec).items():
+        t = random_tensor(name, resolved_shape(d.shape), d.role, seed, device, d.high)
+        out[name] = t if d.role == "int_table" else t.to(dtype)
+    return out
 
 
 def write_random_model(model_dir: str, config: dict, seed: int, dtype=torch.float32) -> str:
