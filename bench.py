@@ -2,10 +2,11 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
     python bench.py --workload smollm2-360m|smollm2-135m [--workload-dtypes bfloat16,float32]
-    python bench.py --design garodra|fusazen|gemosun|renitar [--design-sizes 2048,1024]          (its own JSON line: that design's prefill and
+    python bench.py --design garodra|fusazen|gemosun|renitar|zomurax [--design-sizes 2048,1024]  (its own JSON line: that design's prefill and
                                                                                   decode beside the Llama decoder (renitar: beside the
-                                                                                  Fusazen design) at equal size; garodra also has the
-                                                                                  size 2048-looped)
+                                                                                  Fusazen design, zomurax: beside the Garodra design) at
+                                                                                  equal size; garodra also has the size 2048-looped,
+                                                                                  zomurax the size 2048-full)
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and context 4096 (a
 "step" is one decode step of the whole batch), timed on the device with CUDA events around
@@ -341,6 +342,30 @@ RENITAR_SIZES = {
 }
 
 
+# --design zomurax: the Zomurax design at sizes that resemble a real model's layers, beside the Garodra design (the closest
+# of the library's models: attention through a latent, routed experts of the same form) at equal width and depth.  Eight
+# layers that alternate the two mixers: attention of grouped queries (unit-size q and k, a bias by distance, a sink, a
+# temperature, values mixed with the first layer's) and latent attention over a window; every layer has routed experts
+# (eight, two a token, by the token's id) and one beside them that every token runs.  The latent layers' window is 1,024
+# positions, or ("-full") spans the whole context, so that they read as many positions as the other model's.
+def zomurax_config(width, heads, kv_heads, dim, rot_dim, kv_rank, experts, top, expert_ff, shared, vocab, window, layers=8):
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "v_mix": True,
+           "q_temp": {"coef": 0.2, "every": 1024}}
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5,
+           "rot": {"base": 10000.0, "dims": rot_dim}, "mask": {"size": window}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+    kinds = [("attention", att), ("latent_attention", lat)]
+    return {"architecture": "Zomurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "logit_softcap": 50.0,
+            "layers": [{"type": kinds[i % 2][0], "mixer": kinds[i % 2][1], "mlp": moe} for i in range(layers)]}
+
+
+ZOMURAX_SIZES = {
+    "2048": (zomurax_config(2048, 16, 4, 128, 64, 512, 8, 2, 2048, 2048, 49152, 1024), DESIGN_SIZES["2048"][0], "garodra"),
+    "2048-full": (zomurax_config(2048, 16, 4, 128, 64, 512, 8, 2, 2048, 2048, 49152, 8192), DESIGN_SIZES["2048"][0], "garodra"),
+    "1024": (zomurax_config(1024, 8, 2, 64, 32, 256, 8, 2, 1024, 1024, 49152, 1024), DESIGN_SIZES["1024"][0], "garodra"),
+}
+
+
 class KernelTimes:
     """Device time per entry point of ops.kernels inside real steps (CUDA events around every call; steps run launch
     by launch while this is on, so the figures are shares of a step, not a benchmark of it)."""
@@ -348,7 +373,8 @@ class KernelTimes:
              "latent_prepare", "latent_q_rotate", "attention_latent", "delta_step", "delta_finish", "moe_route",
              "moe_experts_streamed", "moe_experts_grouped", "conv_add", "qkv_prepare", "attention_maps", "diff_combine",
              "gdelta_prepare", "dplr_recurrence", "activate", "layernorm", "depth_mix", "pool_rows", "gate_rows", "tanh_rows",
-             "channel_decay", "rows_silu", "decay_recurrence", "normed_pair", "stream_axpy_norm", "moe_identity_add")
+             "channel_decay", "rows_silu", "decay_recurrence", "normed_pair", "stream_axpy_norm", "moe_identity_add",
+             "qkv_unit_prepare", "latent_prepare_direct", "moe_table", "stream_postnorm", "softcap_rows")
 
     def __init__(self):
         self.spans, self.saved = [], {}
@@ -391,7 +417,8 @@ def design_run(name, steps, warmup, batch, context, tokens, sizes):
     import torch
     import llmi_b200 as L
     from llmi_b200 import SequenceStep
-    tables = {"garodra": DESIGN_SIZES, "fusazen": FUSAZEN_SIZES, "gemosun": GEMOSUN_SIZES, "renitar": RENITAR_SIZES}
+    tables = {"garodra": DESIGN_SIZES, "fusazen": FUSAZEN_SIZES, "gemosun": GEMOSUN_SIZES, "renitar": RENITAR_SIZES,
+              "zomurax": ZOMURAX_SIZES}
     if name not in tables:
         print(f"bench.py: unknown design {name!r}")
         return 2
@@ -462,9 +489,9 @@ def main():
     ap.add_argument("--kv-heads", type=int, default=None,
                     help="with --only: another number of key/value heads (grouped queries), to profile their kernels")
     ap.add_argument("--design", default=None,
-                    help="'garodra', 'fusazen', 'gemosun' or 'renitar': that design's prefill and decode throughput at layer sizes of a real model, beside the "
-                         "Llama decoder (renitar: beside the Fusazen design) at equal size (its own JSON line; the default workload is untouched)")
-    ap.add_argument("--design-sizes", default="2048,1024", help="with --design: which of " + ", ".join(sorted(set(DESIGN_SIZES) | set(GEMOSUN_SIZES))))
+                    help="'garodra', 'fusazen', 'gemosun', 'renitar' or 'zomurax': that design's prefill and decode throughput at layer sizes of a real model, beside the "
+                         "Llama decoder (renitar: beside the Fusazen design, zomurax: beside the Garodra design) at equal size (its own JSON line; the default workload is untouched)")
+    ap.add_argument("--design-sizes", default="2048,1024", help="with --design: which of " + ", ".join(sorted(set(DESIGN_SIZES) | set(GEMOSUN_SIZES) | set(ZOMURAX_SIZES))))
     args = ap.parse_args()
 
     if args.design:

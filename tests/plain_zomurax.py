@@ -58,8 +58,8 @@ def temperature(pos, coef, every):
 
 
 def distance_bias(dist, r1, r2):
-    """What a key ``dist`` positions back loses of its score."""
-    return r1 * math.log(1.0 + r2 * dist)
+    """What a key ``dist`` positions back loses of its score (``dist`` may be an array)."""
+    return r1 * np.log(1.0 + r2 * dist)
 
 
 def in_window(i, j, size):
@@ -68,6 +68,7 @@ def in_window(i, j, size):
 
 
 def mix_values(v, first, lam):
+    """Whole projected rows, all heads at once."""
     return (1.0 - lam) * v + lam * first
 
 
@@ -80,8 +81,8 @@ def attention(m, w, p, x, eps, first_values):
     T = x.shape[0]
     q = rms_unit((x @ w[p + "q"].T).reshape(T, H, dk), eps)
     k = rms_unit((x @ w[p + "k"].T).reshape(T, G, dk), eps)
-    own = (x @ w[p + "v"].T).reshape(T, G, dv)
-    v = own if first_values is None else mix_values(own, first_values, float(w[p + "vmix"]))
+    own = x @ w[p + "v"].T
+    v = (own if first_values is None else mix_values(own, first_values, float(w[p + "vmix"]))).reshape(T, G, dv)
     if m.get("q_temp"):
         q = q * np.array([temperature(t, float(m["q_temp"]["coef"]), float(m["q_temp"]["every"])) for t in range(T)])[:, None, None]
     o = np.zeros((T, H, dv))
@@ -89,7 +90,7 @@ def attention(m, w, p, x, eps, first_values):
         for a in range(H):
             g = a // (H // G)
             s = (k[:i + 1, g] @ q[i, a]) * float(m["scale"])
-            s = s - np.array([distance_bias(i - j, float(w[p + "r1"][a]), float(w[p + "r2"][a])) for j in range(i + 1)])
+            s = s - distance_bias(i - np.arange(i + 1.0), float(w[p + "r1"][a]), float(w[p + "r2"][a]))
             o[i, a] = softmax(s, float(w[p + "sink"][a])) @ v[:i + 1, g]
     return o.reshape(T, H * dv) @ w[p + "o"].T, own
 
