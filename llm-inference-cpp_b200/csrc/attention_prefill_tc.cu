@@ -177,7 +177,6 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const uint32_t o_done = bars + 8u * (5 + 2 * STAGES);
   const uint32_t tmem_slot = o_done + 8u;
 
-  pdl_launch_dependents();
   // The head is the FAST grid index and the job the slow one: blocks start in the order of their linear index, and a
   // long job that starts late is the kernel's tail (with the head as the slow index the longest job of the last head
   // started when the kernel was half over: 51 us for 2,048 tokens x 32 heads against 33 us this way).
@@ -261,6 +260,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   uint32_t tmem;
   asm volatile("ld.shared.u32 %0, [%1];" : "=r"(tmem) : "r"(tmem_slot));
+  // only now: a kernel after this one that started before this block has its tensor memory could take it and then wait
+  // for this block to end (a block that found no work above lets it start by returning)
+  pdl_launch_dependents();
   const uint32_t tmem_s = tmem, tmem_o = tmem + 128;
 
   if (warp == 0) {
