@@ -637,7 +637,10 @@ static int ft_launch_b(const CUtensorMap& mq, const CUtensorMap& mk, const CUten
 template <int HD>
 static int ft_launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkp,
                      const CUtensorMap& mvp, const PrefillTcParams& p, dim3 grid, cudaStream_t stream) {
-  return p.r1 ? ft_launch_b<HD, true>(mq, mk, mv, mkp, mvp, p, grid, stream) : ft_launch_b<HD, false>(mq, mk, mv, mkp, mvp, p, grid, stream);
+  if (p.r1) return ft_launch_b<HD, true>(mq, mk, mv, mkp, mvp, p, grid, stream);
+  const int rc = ft_launch_b<HD, false>(mq, mk, mv, mkp, mvp, p, grid, stream);
+  pairs_may_start_early = true;
+  return rc;
 }
 }  // namespace llmi
 

@@ -187,6 +187,14 @@ inline bool pdl_enabled(int kind) {
   return (mask & kind) != 0;
 }
 
+// Behind which kernels the products on pairs of SMs (gemm_tc_pair_kernel, a cluster of two with all of the tensor memory)
+// may be launched this way: those of the Llama decoder's prompt step, behind which they have always run so — the RMS
+// norm, the prompt attention, and one another.  Launched early behind the routed experts' weighted sum (2,048 tokens,
+// 4,096 rows, every pair of SMs in use), one pair of the 74 now and then never got past its set-up while the other 73
+// finished, and the stream stood still; launched behind the end of that kernel they do not.  A launcher of such a kernel
+// sets this after its launch; every other launch clears it.
+inline thread_local bool pairs_may_start_early = false;
+
 template <typename... KArgs, typename... Args>
 inline int launch_pdl(int kind, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
                       Args... args) {
@@ -200,6 +208,7 @@ inline int launch_pdl(int kind, void (*kernel)(KArgs...), dim3 grid, dim3 block,
   attr[0].val.programmaticStreamSerializationAllowed = pdl_enabled(kind) ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
+  pairs_may_start_early = false;
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...) == cudaSuccess ? LLMI_OK : LLMI_ERR_LAUNCH;
 }
 

@@ -569,17 +569,17 @@ static int launch_tc_pair(const CUtensorMap& mw, const CUtensorMap& mx, const CU
   cfg.blockDim = dim3(TC_THREADS);
   cfg.dynamicSmemBytes = TP_SMEM;
   cfg.stream = stream;
-  cudaLaunchAttribute attr[1];
+  cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeClusterDimension;
   attr[0].val.clusterDim.x = 2;
   attr[0].val.clusterDim.y = 1;
   attr[0].val.clusterDim.z = 1;
-  // NOT a programmatic dependent launch: the pairs start when the kernel before has ended.  Started early behind the
-  // routed experts' weighted sum (2,048 tokens, 4,096 rows: one pair per pair of SMs), one pair of the 74 now and then
-  // never got past its set-up (tensor memory, cluster barrier) while the other 73 finished, and the stream stood still.
-  // The kernel itself still lets the one behind it start early.
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  const bool early = pairs_may_start_early && pdl_enabled(PDL_GEMM);      // (behind any other kernel: when that has ended)
+  attr[1].val.programmaticStreamSerializationAllowed = early ? 1 : 0;
   cfg.attrs = attr;
-  cfg.numAttrs = 1;
+  cfg.numAttrs = 2;
+  pairs_may_start_early = early;
   return cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel, mw, mx, mo, p, m_tiles, n_tiles, bn, out_tma) == cudaSuccess ? LLMI_OK : LLMI_ERR_LAUNCH;
 }
 
@@ -943,6 +943,7 @@ static int launch_tc_wide(const CUtensorMap& mw, const CUtensorMap& mx, const CU
   attr[1].val.programmaticStreamSerializationAllowed = pdl_enabled(PDL_GEMM) ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
+  pairs_may_start_early = false;
   return cudaLaunchKernelEx(&cfg, gemm_tc_wide_kernel<BN>, mw, mx, mo, p, m_tiles, S, boxed3d, out_tma) == cudaSuccess ? LLMI_OK
                                                                                                                : LLMI_ERR_LAUNCH;
 }

@@ -235,7 +235,12 @@ moe_combine_kernel(const float* __restrict__ ys, const int32_t* __restrict__ ite
 
 
 // ------------------------------------------------------------------------------------------------
-// The grouped products of many items on the 5th-generation tensor cores (tcgen05), for experts without a gate matrix.
+// The grouped products of many items on the 5th-generation tensor cores (tcgen05).
+//
+// Experts with a gate matrix: the up product's weight tile alternates gate and up rows.  It comes so from memory — the
+// tensor map has a dimension of two between the row and the k entries, whose stride is the distance from the gate
+// matrices to the up matrices — so that neighbouring TMEM lanes hold an output's gate and up sums; a shuffle hands each
+// of the two threads both sums of half of the tokens, and act(gate) * up leaves as bf16.
 //
 // The items' input rows are first copied into the order of the grouping (moe_gather_rows_kernel), so that a tile of
 // 128 items of one expert is a box of a 2-d tensor map; the experts' weights [E, N, K] are a 3-d map whose boxes end
@@ -256,7 +261,8 @@ constexpr int GT_TMEM_COLS = 2 * GT_BN;
 
 struct GtParams {
   int N, K;                      // an expert's weight [N, K]
-  void* out;                     // [items, N], row pitch ldo: bf16 act(v) (mode 0) or fp32 v (mode 1)
+  void* out;                     // row pitch ldo: bf16 act(v) [items, N] (mode 0), fp32 v [items, N] (mode 1), or bf16
+                                 // act(gate) * up [items, N / 2] (mode 2: W's rows alternate gate and up rows)
   long ldo;
   int mode, act;                 // act 0: silu, 1: tanh GELU, 2: relu squared, 3: exact GELU
   const int32_t *offsets, *tile_expert, *tile_row0, *n_tiles;
@@ -267,6 +273,13 @@ __device__ __forceinline__ void tma_load_3d_box(uint32_t dst, const CUtensorMap*
   asm volatile(
       "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
       ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2)
+      : "memory");
+}
+
+__device__ __forceinline__ void tma_load_4d_box(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, int c3, uint32_t bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
+      ::"r"(dst), "l"(map), "r"(bar), "r"(c0), "r"(c1), "r"(c2), "r"(c3)
       : "memory");
 }
 
@@ -333,7 +346,8 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
           if (it >= GT_STAGES && !mbar_wait(empty_bar(s), ((it / GT_STAGES) - 1) & 1, p.error_flag, 21)) { ok = false; break; }
           mbar_expect_tx(full_bar(s), GT_STAGE_BYTES);
           const uint32_t a_dst = base + s * GT_STAGE_BYTES;
-          tma_load_3d_box(a_dst, &map_w, i * TC_BK, mt * TC_BM, e, full_bar(s));
+          if (p.mode == 2) tma_load_4d_box(a_dst, &map_w, i * TC_BK, 0, mt * (TC_BM / 2), e, full_bar(s));
+          else tma_load_3d_box(a_dst, &map_w, i * TC_BK, mt * TC_BM, e, full_bar(s));
           tma_load_2d(a_dst + GT_A_BYTES, &map_x, i * TC_BK, row0, full_bar(s));
         }
       }
@@ -385,7 +399,19 @@ moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
           __syncwarp();
           if (lane == 0) mbar_arrive(acc_empty(b));
         }
-        if (m < p.N) {
+        if (p.mode == 2) {
+          // even lanes hold gate sums, odd lanes up sums of the same feature: the even lane finishes the chunk's tokens
+          // 0..7, the odd lane 8..15
+          const bool is_gate = (m & 1) == 0;
+          const int first = c0 + (is_gate ? 0 : 8);
+          __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)(row0 + first) * p.ldo + (m >> 1);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) {
+            const float recv = __shfl_xor_sync(0xffffffffu, is_gate ? v[c + 8] : v[c], 1);
+            const float g = is_gate ? v[c] : recv, u = is_gate ? recv : v[c + 8];
+            if (m < p.N && first + c < n_valid) o[(size_t)c * p.ldo] = __float2bfloat16_rn(gated_value(g, u, p.act));
+          }
+        } else if (m < p.N) {
 #pragma unroll
           for (int c = 0; c < 16; ++c) {
             if (c0 + c >= n_valid) break;
@@ -422,6 +448,15 @@ static int gt_make_map(CUtensorMap* map, const void* ptr, long k, long rows, lon
     if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess)
       return LLMI_ERR_DRIVER;
     fn = (EncodeFn)sym;
+  }
+  if (batch < 0) {      // -batch experts with a gate matrix: [expert][row][gate, up][k], `ld` the bytes from the gate matrices to the up matrices
+    const cuuint64_t dims4[4] = {(cuuint64_t)k, 2, (cuuint64_t)rows, (cuuint64_t)-batch};
+    const cuuint64_t strides4[3] = {(cuuint64_t)ld, (cuuint64_t)k * 2, (cuuint64_t)rows * (cuuint64_t)k * 2};
+    const cuuint32_t box4[4] = {(cuuint32_t)TC_BK, 2, (cuuint32_t)box_rows, 1};
+    const cuuint32_t elem4[4] = {1, 1, 1, 1};
+    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(ptr), dims4, strides4, box4, elem4,
+              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? LLMI_OK : LLMI_ERR_DRIVER;
   }
   const cuuint64_t dims[3] = {(cuuint64_t)k, (cuuint64_t)rows, (cuuint64_t)(batch ? batch : 1)};
   const cuuint64_t strides[2] = {(cuuint64_t)ld * 2, (cuuint64_t)rows * (cuuint64_t)ld * 2};
@@ -466,20 +501,24 @@ LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const 
   int32_t* tile_expert = item_pos + n_items;
   int32_t* tile_row0 = tile_expert + max_tiles;
   int32_t* n_tiles = tile_row0 + max_tiles;
-  // Many items of experts without a gate matrix, at sizes that fill 128 x 128 tiles: the tcgen05 kernel (h_sorted lends
-  // [n_items, W] bf16 for the items' input rows in the grouping's order).  LLMI_MOE_TC=0 keeps the mma.sync tiles.
+  // Many items at sizes that fill 128 x 128 tiles: the tcgen05 kernel (h_sorted lends [n_items, W] bf16 for the items'
+  // input rows in the grouping's order).  Experts with a gate matrix: the up matrices must lie behind the gate matrices
+  // in memory, at a distance of whole 16 bytes.  LLMI_MOE_TC=0 keeps the mma.sync tiles.
   static int tc_ok = -1;
   if (tc_ok < 0) {
     const char* ev = getenv("LLMI_MOE_TC");
     tc_ok = (ev && ev[0] == '0') ? 0 : 1;
   }
-  const bool tc = tc_ok && !wg && h_sorted && error_flag && n_items >= 1024 && W >= 128 && F >= 128 && !((uintptr_t)h_sorted & 15);
+  const long gate_to_up = wg ? (long)((const char*)wu - (const char*)wg) : 0;
+  const bool gate_ok = !wg || (gate_to_up > 0 && gate_to_up % 16 == 0 && gate_to_up < (1L << 39));
+  const bool tc = tc_ok && gate_ok && h_sorted && error_flag && n_items >= 1024 && W >= 128 && F >= 128 && !((uintptr_t)h_sorted & 15);
   int rc = launch_pdl(PDL_SMALL, moe_group_kernel, dim3(1), dim3(1024), 0, stream, idx, n_items, E, offsets, sorted_items, item_pos,
                       tile_expert, tile_row0, n_tiles, tc ? GT_BN : GB_M);
   if (rc != LLMI_OK) return rc;
   if (tc) {
     CUtensorMap mw_up, mx_up, mw_down, mx_down;
-    if ((rc = gt_make_map(&mw_up, wu, W, F, E, W, TC_BM)) != LLMI_OK) return rc;
+    rc = wg ? gt_make_map(&mw_up, wg, W, F, -E, gate_to_up, TC_BM / 2) : gt_make_map(&mw_up, wu, W, F, E, W, TC_BM);
+    if (rc != LLMI_OK) return rc;
     if ((rc = gt_make_map(&mx_up, h_sorted, W, n_items, 0, W, GT_BN)) != LLMI_OK) return rc;
     if ((rc = gt_make_map(&mw_down, wd, F, W, E, F, TC_BM)) != LLMI_OK) return rc;
     if ((rc = gt_make_map(&mx_down, a_sorted, F, n_items, 0, F, GT_BN)) != LLMI_OK) return rc;
@@ -493,8 +532,9 @@ LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const 
                     (const int32_t*)sorted_items, (const int32_t*)(offsets + E), top, W, (__nv_bfloat16*)h_sorted);
     if (rc != LLMI_OK) return rc;
     const int tiles_most = (n_items + GT_BN - 1) / GT_BN + E;
-    const int mt_up = (F + TC_BM - 1) / TC_BM, mt_down = (W + TC_BM - 1) / TC_BM;
-    GtParams pu{F, W, a_sorted, (long)F, 0, act, offsets, tile_expert, tile_row0, n_tiles, error_flag};
+    const int up_rows = wg ? 2 * F : F;
+    const int mt_up = (up_rows + TC_BM - 1) / TC_BM, mt_down = (W + TC_BM - 1) / TC_BM;
+    GtParams pu{up_rows, W, a_sorted, (long)F, wg ? 2 : 0, act, offsets, tile_expert, tile_row0, n_tiles, error_flag};
     GtParams pd{W, F, (void*)y_sorted, (long)W, 1, 0, offsets, tile_expert, tile_row0, n_tiles, error_flag};
     const long sms = sm_count();
     rc = launch_pdl(PDL_GEMM, moe_grouped_tc_kernel, dim3((unsigned)min((long)tiles_most * mt_up, sms)), dim3(TC_THREADS), (size_t)GT_SMEM,

@@ -215,8 +215,8 @@ LLMI_EXPORT int llmi_embed(int dtype, const void* table, const int32_t* ids, flo
   return launch_status();
 }
 
-LLMI_EXPORT int llmi_rmsnorm(int out_dtype, const float* x, const float* weight, void* out, const int32_t* rows,
-                             int n_rows, int width, float eps, cudaStream_t stream) {
+static int launch_rmsnorm(int out_dtype, const float* x, const float* weight, void* out, const int32_t* rows, int n_rows, int width,
+                          float eps, cudaStream_t stream) {
   if (n_rows <= 0 || width <= 0) return LLMI_ERR_BAD_SIZE;
   const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
   if (out_dtype != LLMI_DTYPE_F32 && out_dtype != LLMI_DTYPE_BF16) return LLMI_ERR_BAD_DTYPE;
@@ -238,7 +238,13 @@ LLMI_EXPORT int llmi_rmsnorm(int out_dtype, const float* x, const float* weight,
     return launch_pdl(PDL_SMALL, rmsnorm_kernel<float>, n_rows, threads, 0, stream, x, weight, (float*)out, rows, width, eps);
   else
     return launch_pdl(PDL_SMALL, rmsnorm_kernel<__nv_bfloat16>, n_rows, threads, 0, stream, x, weight, (__nv_bfloat16*)out, rows, width, eps);
-  return launch_status();
+}
+
+LLMI_EXPORT int llmi_rmsnorm(int out_dtype, const float* x, const float* weight, void* out, const int32_t* rows,
+                             int n_rows, int width, float eps, cudaStream_t stream) {
+  const int rc = launch_rmsnorm(out_dtype, x, weight, out, rows, n_rows, width, eps, stream);
+  pairs_may_start_early = true;
+  return rc;
 }
 
 // Streaming multiprocessors of the current device, for dispatch rules that live on the host side of the library.

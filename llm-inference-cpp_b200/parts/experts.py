@@ -102,8 +102,10 @@ class RoutedExperts:
             router = torch.cat([router, tensors["shared.sg"].reshape(1, self.width)], dim=0)
             self.w_shared_up, self.w_shared_down = rt.to_compute(tensors["shared.up"]), rt.to_compute(tensors["shared.down"])
         self.w_router = rt.to_compute(router) if router is not None else None
-        self.w_gate = rt.to_compute(torch.stack([tensors[f"e{i}.gate"] for i in range(self.E)])) if self.gated else None
-        self.w_up = rt.to_compute(torch.stack([tensors[f"e{i}.up"] for i in range(self.E)]))
+        # [gate | up][expert][inner][width] in one piece: the grouped tcgen05 tiles read gate and up rows in turn from it
+        both = rt.to_compute(torch.stack([tensors[f"e{i}.{n}"] for n in (("gate", "up") if self.gated else ("up",)) for i in range(self.E)]))
+        self.w_gate = both[:self.E] if self.gated else None
+        self.w_up = both[self.E:] if self.gated else both
         self.w_down = rt.to_compute(torch.stack([tensors[f"e{i}.down"] for i in range(self.E)]))
 
     def weight_bytes(self) -> int:

@@ -536,3 +536,47 @@ def test_capped_rows_and_experts_by_the_tokens_id():
     live = torch.arange(35, device="cuda:0") != 4
     assert torch.equal(idx[live], table[ids[live].long()]) and (idx[4] == -1).all() and (wt[4] == 0).all()
     assert torch.allclose(wt[live], torch.full((34, 3), 1 / 3, device="cuda:0"))
+
+
+@pytest.mark.parametrize("act", ["silu", "gelu_tanh"])
+@pytest.mark.parametrize("T,E,top,W,F", [(3, 4, 2, 64, 48), (300, 5, 3, 136, 72), (600, 4, 2, 128, 128), (1500, 8, 2, 256, 200), (1024, 3, 1, 192, 136), (700, 12, 3, 512, 64)])
+def test_gated_experts_on_every_kind_of_tile(T, E, top, W, F, act):
+    """Streamed weights (a few tokens), mma.sync tiles, tcgen05 tiles (from 1,024 items and 128 rows on, gate and up rows in
+    turn): the same sum, with token rows of no sequence and one expert that nobody picks; rows of the up matrices that lie
+    ahead of the gate matrices in memory take the other tiles."""
+    import torch
+    from llmi_b200.engine.runtime import Runtime
+    from llmi_b200.ops import kernels
+    rt = Runtime(torch.bfloat16, "cuda:0")
+    gen = torch.Generator(device="cuda:0").manual_seed(T + E)
+
+    def rnd(*shape, gain=1.0):
+        return (torch.randn(*shape, generator=gen, device="cuda:0") * gain).to(torch.bfloat16)
+    h, both, wd = rnd(T, W), rnd(2, E, F, W, gain=2 * W ** -0.5), rnd(E, W, F, gain=F ** -0.5)
+    score = torch.rand(T, E, generator=gen, device="cuda:0")
+    if E > top:
+        score[:, E - 2] = -1.0                                            # nobody picks it
+    idx = score.topk(top, dim=1).indices.to(torch.int32).contiguous()
+    idx[T // 2] = -1
+    wt = torch.full((T, top), 1.0 / top, device="cuda:0")
+    code = kernels.EXPERT_ACTIVATIONS[act]
+    fn = torch.nn.functional.silu if act == "silu" else lambda z: torch.nn.functional.gelu(z, approximate="tanh")
+    for wg, wu in ((both[0], both[1]), (both[1], both[0])):
+        y = torch.full((T, W), float("nan"), device="cuda:0")
+        if kernels.moe_grouped_applies(h, W, F, E):
+            kernels.moe_experts_grouped(h, wg, wu, wd, idx, wt, code, rt, y)
+            again = torch.ones((T, W), device="cuda:0")
+            kernels.moe_experts_grouped(h, wg, wu, wd, idx, wt, code, rt, again, add=True)
+            assert torch.equal(again, 1.0 + y)
+        else:
+            kernels.moe_experts_streamed(h, wg, wu, wd, idx, wt, code, torch.empty((T, top, F), device="cuda:0"), y)
+        kernels.check_device_errors(torch.device("cuda:0"))
+        hd, ref = h.double(), torch.zeros((T, W), dtype=torch.float64, device="cuda:0")
+        for e in range(E):
+            for j in range(top):
+                rows = (idx[:, j] == e).nonzero().flatten()
+                if rows.numel():
+                    a = fn(hd[rows] @ wg[e].double().T) * (hd[rows] @ wu[e].double().T)
+                    ref[rows] += wt[rows, j].double()[:, None] * (a @ wd[e].double().T)
+        err = (y.double() - ref).abs().max(dim=1).values / ref.abs().max()
+        assert torch.isfinite(y).all() and float(err.max()) < 1.5e-2 and float(y[T // 2].abs().max()) == 0.0, (int(err.argmax()), float(err.max()))
