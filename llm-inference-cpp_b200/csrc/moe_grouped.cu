@@ -26,18 +26,36 @@ constexpr int GB_M = 64, GB_N = 64, GB_K = 64, GB_LD = GB_K + 8, GB_STAGES = 3;
 constexpr int GB_CH = GB_K / 8;            // 16-byte pieces of a tile row
 constexpr int GB_SLOTS = GB_M * GB_CH / 128;   // pieces a thread copies per operand and stage
 
+// Where a table gives the token's experts by its id (no router): the grouping kernel looks them up itself and leaves the
+// choices and their equal weights as the router's kernel would (llmi_moe_table is the same for a handful of tokens).
+struct GroupTable {
+  const int32_t* table;         // [vocab, top], null: idx holds the choices
+  const int32_t *token_ids, *tok_seq;
+  int vocab, top;
+  float* wt;
+};
+
 // meta: [0] number of tiles; offsets [E + 1]; tile_expert, tile_row0 [max_tiles]
 __global__ void __launch_bounds__(1024)
-moe_group_kernel(const int32_t* __restrict__ idx, int n_items, int E, int32_t* __restrict__ offsets,
+moe_group_kernel(int32_t* idx, int n_items, int E, int32_t* __restrict__ offsets,
                  int32_t* __restrict__ sorted_items, int32_t* __restrict__ item_pos, int32_t* __restrict__ tile_expert,
-                 int32_t* __restrict__ tile_row0, int32_t* __restrict__ n_tiles, int tile_rows) {
+                 int32_t* __restrict__ tile_row0, int32_t* __restrict__ n_tiles, int tile_rows, GroupTable by_id) {
   __shared__ int cnt[256], cursor[256];
   pdl_wait();
   pdl_launch_dependents();
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
   for (int i = threadIdx.x; i < n_items; i += blockDim.x) {
-    const int e = idx[i];
+    int e;
+    if (by_id.table) {
+      const int t = i / by_id.top, id = by_id.token_ids[t];
+      const bool live = by_id.tok_seq[t] >= 0 && id >= 0 && id < by_id.vocab;
+      e = live ? by_id.table[(size_t)id * by_id.top + (i - t * by_id.top)] : -1;
+      idx[i] = e;                                        // (this thread reads it again below)
+      by_id.wt[i] = live ? 1.0f / (float)by_id.top : 0.f;
+    } else {
+      e = idx[i];
+    }
     if (e >= 0) atomicAdd(&cnt[e], 1);
   }
   __syncthreads();
@@ -479,12 +497,14 @@ LLMI_EXPORT long llmi_moe_group_ints(int n_items, int E) {
   return (E + 1) + 2L * n_items + 2 * max_tiles + 1;
 }
 
+// table (optional, int32 [vocab, top]): idx and wt are not given but made here from the tokens' ids (GroupTable).
 // id_wt (optional, fp32 [n_tokens]): a token's summed weight of chosen experts that hand their input on (choices of
 // index -1): id_wt[t] * h[t] joins the token's sum in the kernel that forms it.
 LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const void* wu, const void* wd, int W, int F, int E,
-                                 int top, const int32_t* idx, const float* wt, int act, int32_t* scratch, long scratch_ints,
+                                 int top, int32_t* idx, float* wt, int act, int32_t* scratch, long scratch_ints,
                                  void* a_sorted, float* y_sorted, float* y, long ldy, int n_tokens, int add, void* h_sorted,
-                                 int* error_flag, const float* id_wt, cudaStream_t stream) {
+                                 int* error_flag, const float* id_wt, const int32_t* table, int vocab, const int32_t* token_ids,
+                                 const int32_t* tok_seq, cudaStream_t stream) {
   if (n_tokens <= 0 || W <= 0 || F <= 0 || E <= 0 || E > 256 || top <= 0) return LLMI_ERR_BAD_SIZE;
   if ((W % 8) || (F % 8) || (ldh % 8) || ((uintptr_t)h & 15) || ((uintptr_t)wg & 15) || ((uintptr_t)wu & 15) || ((uintptr_t)wd & 15) ||
       ((uintptr_t)a_sorted & 15))
@@ -513,7 +533,7 @@ LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const 
   const bool gate_ok = !wg || (gate_to_up > 0 && gate_to_up % 16 == 0 && gate_to_up < (1L << 39));
   const bool tc = tc_ok && gate_ok && h_sorted && error_flag && n_items >= 1024 && W >= 128 && F >= 128 && !((uintptr_t)h_sorted & 15);
   int rc = launch_pdl(PDL_SMALL, moe_group_kernel, dim3(1), dim3(1024), 0, stream, idx, n_items, E, offsets, sorted_items, item_pos,
-                      tile_expert, tile_row0, n_tiles, tc ? GT_BN : GB_M);
+                      tile_expert, tile_row0, n_tiles, tc ? GT_BN : GB_M, GroupTable{table, token_ids, tok_seq, vocab, top, wt});
   if (rc != LLMI_OK) return rc;
   if (tc) {
     CUtensorMap mw_up, mx_up, mw_down, mx_down;
@@ -544,7 +564,7 @@ LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const 
                     (size_t)GT_SMEM, stream, mw_down, mx_down, pd, mt_down);
     if (rc != LLMI_OK) return rc;
     return launch_pdl(PDL_SMALL, moe_combine_kernel, dim3(n_tokens, combine_cuts), dim3(256), 0, stream, (const float*)y_sorted,
-                      (const int32_t*)item_pos, wt, top, W, y, ldy, add, (const __nv_bfloat16*)h, ldh, id_wt);
+                      (const int32_t*)item_pos, (const float*)wt, top, W, y, ldy, add, (const __nv_bfloat16*)h, ldh, id_wt);
   }
   const size_t smem_up = (size_t)GB_STAGES * 3 * GB_M * GB_LD * 2, smem_down = (size_t)GB_STAGES * 2 * GB_M * GB_LD * 2;
   const __nv_bfloat16* hb = (const __nv_bfloat16*)h;
@@ -583,7 +603,7 @@ LLMI_EXPORT int llmi_moe_grouped(const void* h, long ldh, const void* wg, const 
                   (const int32_t*)tile_row0, (const int32_t*)n_tiles, (void*)y_sorted, (long)W, 0, 0L, 0L);
   if (rc != LLMI_OK) return rc;
   return launch_pdl(PDL_SMALL, moe_combine_kernel, dim3(n_tokens, combine_cuts), dim3(256), 0, stream, (const float*)y_sorted,
-                    (const int32_t*)item_pos, wt, top, W, y, ldy, add, (const __nv_bfloat16*)h, ldh, id_wt);
+                    (const int32_t*)item_pos, (const float*)wt, top, W, y, ldy, add, (const __nv_bfloat16*)h, ldh, id_wt);
 }
 
 // `batch` products of equal sizes on the tensor cores (bf16), one per head: out[:, b*by : b*by+N] = x[:, b*bx : b*bx+K] . w[b]^T,

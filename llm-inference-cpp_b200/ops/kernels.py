@@ -1560,11 +1560,15 @@ def moe_grouped_applies(h: torch.Tensor, W: int, F: int, E: int) -> bool:
 
 
 def moe_experts_grouped(h: torch.Tensor, w_gate, w_up, w_down, idx, wt, act: int, rt, y: torch.Tensor, add: bool = False,
-                        id_wt: torch.Tensor | None = None) -> None:
+                        id_wt: torch.Tensor | None = None, by_id=None) -> None:
     """The same result as :func:`moe_experts_streamed` for many tokens: the (token, choice) items are grouped by expert
     and each expert's products run as tensor-core tiles over its rows.  bf16; ``rt`` lends the scratch.  ``id_wt`` (fp32
-    [T], optional): id_wt[t] * h[t] joins token t's sum (what :func:`moe_identity_add` adds, without a kernel of its own)."""
-    _need_cuda(h, w_gate, w_up, w_down, idx, wt, y, id_wt)
+    [T], optional): id_wt[t] * h[t] joins token t's sum (what :func:`moe_identity_add` adds, without a kernel of its own).
+    ``by_id`` = (table, token_ids, ctx): ``idx`` and ``wt`` are not read but made here as :func:`moe_table` makes them."""
+    table, token_ids, ctx = by_id if by_id is not None else (None, None, None)
+    _need_cuda(h, w_gate, w_up, w_down, idx, wt, y, id_wt, table, token_ids)
+    assert table is None or (table.dtype == token_ids.dtype == torch.int32 and table.is_contiguous() and table.shape[1] == idx.shape[1]
+                             and token_ids.shape[0] == h.shape[0])
     assert id_wt is None or (id_wt.dtype == torch.float32 and id_wt.is_contiguous() and id_wt.numel() >= h.shape[0])
     T, W = h.shape
     E, F, _ = w_up.shape
@@ -1582,7 +1586,8 @@ def moe_experts_grouped(h: torch.Tensor, w_gate, w_up, w_down, idx, wt, act: int
     _check("moe_grouped", lib().llmi_moe_grouped(
         _ptr(h), c_long(h.stride(0)), _ptr(w_gate), _ptr(w_up), _ptr(w_down), c_int(W), c_int(F), c_int(E), c_int(top), _ptr(idx),
         _ptr(wt), c_int(act), _ptr(scratch), c_long(n_int), _ptr(a_sorted), _ptr(y_sorted), _ptr(y), c_long(y.stride(0)), c_int(T),
-        c_int(1 if add else 0), _ptr(h_sorted), _ptr(tc_scratch(h.device).error), _ptr(id_wt), _stream()))
+        c_int(1 if add else 0), _ptr(h_sorted), _ptr(tc_scratch(h.device).error), _ptr(id_wt), _ptr(table),
+        c_int(table.shape[0] if table is not None else 0), _ptr(token_ids), _ptr(ctx.tok_seq if ctx is not None else None), _stream()))
 
 
 # ---------------------------------------------------------------------------------------------

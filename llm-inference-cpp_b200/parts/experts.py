@@ -120,16 +120,19 @@ class RoutedExperts:
         idx = rt.scratch("router_choice", (T, self.top), torch.int32)
         wt = rt.scratch("router_weight", (T, self.top), torch.float32)
         id_wt = rt.scratch("router_identity", (T,), torch.float32) if self.identity else None
+        grouped = kernels.moe_grouped_applies(h, self.width, self.inner, self.E)
         if self.table is not None:
-            kernels.moe_table(self.table, ctx.token_ids, ctx, idx, wt)
+            if not grouped:      # (the grouping kernel looks the table up itself)
+                kernels.moe_table(self.table, ctx.token_ids, ctx, idx, wt)
         else:
             logits = rt.scratch("router_logits", (T, self.w_router.shape[0]), torch.float32)
             kernels.linear(h, self.w_router, logits, None, kernels.OUT_STORE_F32)
             kernels.moe_route(logits, self.top, ctx, idx, wt, self.route_mode, self.n_groups, self.keep, experts=self.n_out,
                               correction=self.correction, scale=self.route_scale, identity=self.identity, id_wt=id_wt)
-        if kernels.moe_grouped_applies(h, self.width, self.inner, self.E):
+        if grouped:
             # (what the chosen experts without tensors add — the token's input times their summed weight — joins the sum there)
-            kernels.moe_experts_grouped(h, self.w_gate, self.w_up, self.w_down, idx, wt, self.act, rt, x, add=not store, id_wt=id_wt)
+            kernels.moe_experts_grouped(h, self.w_gate, self.w_up, self.w_down, idx, wt, self.act, rt, x, add=not store, id_wt=id_wt,
+                                        by_id=None if self.table is None else (self.table, ctx.token_ids, ctx))
         else:
             a = rt.scratch("experts_act", (T, self.top, self.inner), torch.float32)
             kernels.moe_experts_streamed(h, self.w_gate, self.w_up, self.w_down, idx, wt, self.act, a, x, add=not store)
