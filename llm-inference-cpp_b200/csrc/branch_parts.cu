@@ -218,7 +218,10 @@ LLMI_EXPORT int llmi_stream_postnorm(float* x, const float* y, float alpha, int 
                                      void* h, cudaStream_t stream) {
   if (n_rows <= 0 || W <= 0 || (y == nullptr) != (norm_w == nullptr) || (!y && !h)) return LLMI_ERR_BAD_SIZE;
   if (W % 4 == 0 && (((uintptr_t)x & 15) || ((uintptr_t)y & 15) || ((uintptr_t)norm_w & 15) || ((uintptr_t)h & 15))) return LLMI_ERR_ALIGN;
-  const int threads = W >= 2048 ? 512 : (W >= 1024 ? 256 : (W >= 256 ? 128 : 64));
+  // few rows: as many threads as a row gives work, for the shortest way through; many: four pieces a thread and more rows at a time
+  const int few = W >= 2048 ? 512 : (W >= 1024 ? 256 : (W >= 256 ? 128 : 64));
+  const int many = W >= 8192 ? 512 : (W >= 4096 ? 256 : (W >= 2048 ? 128 : 64));
+  const int threads = n_rows >= 512 ? many : few;
   if (!h || dtype == LLMI_DTYPE_F32)
     return launch_pdl(PDL_SMALL, stream_postnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, x, y, alpha, W, norm_w, eps,
                       (float*)h);

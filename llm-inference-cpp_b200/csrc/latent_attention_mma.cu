@@ -278,7 +278,7 @@ attention_latent_mma_kernel(const LatentMmaArgs a) {
           for (int c = threadIdx.x; c < a.C; c += blockDim.x) a.out[(size_t)t * a.ldo + (size_t)hh * a.C + c] = __float2bfloat16_rn(0.f);
 }
 
-// One block per (token, head): joins the cuts.  out = sum_s e^(m_s - M) O_s / sum_s e^(m_s - M) l_s.  The weights
+// One block per (token, head) and 128 columns: joins the cuts.  out = sum_s e^(m_s - M) O_s / sum_s e^(m_s - M) l_s.  The weights
 // e^(m_s - M) / denominator are made once, in shared memory; every thread then adds its columns over the cuts with
 // independent loads.
 constexpr int LM_MAX_SPLITS = 512;
@@ -305,7 +305,7 @@ attention_latent_join_kernel(const float* __restrict__ ws_o, const float* __rest
   const float denom = block_sum(part, red);
   const float inv = 1.0f / denom;
   const float* o = ws_o + (size_t)item * splits * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
     float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
     int s = 0;
     for (; s + 4 <= splits; s += 4) {
@@ -385,6 +385,6 @@ LLMI_EXPORT int llmi_attention_latent_mma(const void* qa, long ldq, void* out, l
   }
   if (rc != LLMI_OK || splits == 1) return rc;
   const long items = (long)n_tokens * n_heads;
-  return launch_pdl(PDL_SMALL, attention_latent_join_kernel, dim3((unsigned)items), dim3(128), 0, stream, (const float*)a.ws_o,
+  return launch_pdl(PDL_SMALL, attention_latent_join_kernel, dim3((unsigned)items, (C + 127) / 128), dim3(128), 0, stream, (const float*)a.ws_o,
                     (const float*)a.ws_ml, (__nv_bfloat16*)out, ldo, tok_seq, n_heads, C, splits);
 }
