@@ -236,7 +236,9 @@ __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ ys, const int32_t* __restrict__ item_pos, const float* __restrict__ wt, int top,
                    int W, float* __restrict__ y, long ldy, int add, const __nv_bfloat16* __restrict__ h, long ldh,
                    const float* __restrict__ id_wt) {
-  pdl_launch_dependents();
+  // Beyond a handful of tokens a product in clusters of blocks may follow: those start when this kernel has ended (see
+  // pairs_may_start_early).
+  if (gridDim.x <= 16) pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const float idw = id_wt ? id_wt[t] : 0.f;          // what the token's chosen experts that hand their input on weigh together
