@@ -90,6 +90,9 @@ constexpr int ACT_STORE_RELU2 = 2;
 // and mode 6: a plain store (bias added) through the exact GELU, v * Phi(v) (OUT_STORE with `act` = 3).
 constexpr int OUT_GELU_REQUEST = 6;
 constexpr int ACT_STORE_GELU = 3;
+// and mode 7: the gated epilogue of OUT_SWIGLU with the bounded gate (OUT_SWIGLU with `act` = ACT_BOUNDED and two constants).
+constexpr int OUT_BOUNDED_REQUEST = 7;
+constexpr int ACT_BOUNDED = 4;
 // What a storing epilogue writes for the value v (bias added): v, relu(v)^2 or 0.5 v (1 + erf(v / sqrt(2))) as `act` says.
 __device__ __forceinline__ float stored_value(float v, int act) {
   if (act == ACT_STORE_RELU2) {
@@ -119,6 +122,23 @@ __device__ __forceinline__ float gated_value(float g, float u, int act) {
   const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
   const float th = 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * z));
   return 0.5f * g * (1.0f + th) * u;
+}
+
+// The bounded gate: g from above at `limit`, u between -limit and limit;  g * logistic(alpha g) * (u + 1).
+__device__ __forceinline__ float bounded_gate(float g, float u, float alpha, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+// The gated epilogues' value with the constants of the activations that have any (the fast exponential and divide again).
+struct GateConstants {
+  float alpha, limit;           // ACT_BOUNDED
+};
+__device__ __forceinline__ float gated_value(float g, float u, int act, const GateConstants& c) {
+  if (act != ACT_BOUNDED) return gated_value(g, u, act);
+  g = fminf(g, c.limit);
+  u = fminf(fmaxf(u, -c.limit), c.limit);
+  return __fdividef(g, 1.0f + __expf(-c.alpha * g)) * (u + 1.0f);
 }
 
 // Facts and one-time set-up per device.  A process may drive several GPUs, and a function attribute (the

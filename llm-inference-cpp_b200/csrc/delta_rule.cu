@@ -12,6 +12,10 @@
 //   llmi_delta_recurrence   per (sequence, head, slice of columns): the recurrence over the step's tokens
 //   llmi_delta_finish       per (token, head): o / rms(o) * w * act(gate) in the compute type (parallel over tokens)
 // The input `proj` is one fp32 row per token: [ q (Hk*D) | k (Hk*D) | v (H*Dv) | b (H) | a (H) | gate (H*Dv) ].
+// With `channel` the decay has a number per key channel instead of one per head: g in (0, 1) multiplies row d of S with
+// its own factor, g[d] = exp(-exp(A_log_h) * softplus(z[d] + dt_bias[d])), with z [T, H*D] made beforehand (a low-rank path
+// of the layer's input), and the input rows are [ q | k | v | b (H) | ... ].  Steps of single tokens have kernels of
+// their own for that form (channel_delta.cu).
 // The recurrence treats a column of S alone, and a step only continues what the slab holds: the result does not
 // depend on how a prompt was cut or on what else is in the batch.
 #include <math.h>
@@ -24,6 +28,11 @@ constexpr int DELTA_MAX_TAPS = 16;
 
 struct DeltaDims {
   int H, Hk, D, Dv, taps;
+  int channel = 0;                                       // a decay per key channel
+  // where a prepared row keeps the decays and the write strengths: [ q^ | k^ | v | beta | decay ], with `channel`
+  // [ q^ | k^ | v | decay (H*D) | beta (H) ] (the decays on a 16-byte boundary where the sizes allow it)
+  __host__ __device__ int decay_at() const { return channel ? n_conv() : n_conv() + H; }
+  __host__ __device__ int beta_at() const { return channel ? n_conv() + H * D : n_conv(); }
   __host__ __device__ int n_qk() const { return 2 * Hk * D; }
   __host__ __device__ int n_conv() const { return 2 * Hk * D + H * Dv; }
   __host__ __device__ long state_floats() const { return (long)H * D * Dv + (long)(taps - 1) * n_conv(); }
@@ -35,7 +44,7 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 
 // One block per (token, piece).  Pieces 0 .. 2 Hk - 1: one head of q or k (convolution, silu, unit norm); the pieces
 // behind them: 256 channels of v each (convolution, silu); the last piece also makes beta and decay of every head.
-// prep: fp32 [T, Nc + 2H]: [ q^ | k^ | v | beta | decay ].
+// prep: fp32 [T, Nc + 2H]: [ q^ | k^ | v | beta | decay ]; with `channel` [T, Nc + H*D + H] and further pieces, 256 decays each.
 constexpr int DELTA_V_PIECE = 256;
 
 __device__ __forceinline__ float delta_conv_one(const float* __restrict__ proj, long ld, const float* __restrict__ carry,
@@ -55,7 +64,7 @@ delta_prepare_kernel(const float* __restrict__ proj, long ld, DeltaDims m, const
                      const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ state,
                      const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos,
                      const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_slot,
-                     float* __restrict__ prep, long ldp) {
+                     float* __restrict__ prep, long ldp, const float* __restrict__ z, long ldz) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -84,15 +93,20 @@ delta_prepare_kernel(const float* __restrict__ proj, long ld, DeltaDims m, const
     for (int d = threadIdx.x; d < m.D; d += blockDim.x) out[base + d] *= sc;
     return;
   }
-  const int vp = piece - 2 * m.Hk, n_v = m.H * m.Dv;
+  const int vp = piece - 2 * m.Hk, n_v = m.H * m.Dv, v_pieces = (n_v + DELTA_V_PIECE - 1) / DELTA_V_PIECE;
+  if (vp >= v_pieces) {                                  // (channel only) the decays
+    const int c0 = (vp - v_pieces) * DELTA_V_PIECE;
+    for (int c = c0 + threadIdx.x; c < min(m.H * m.D, c0 + DELTA_V_PIECE); c += blockDim.x)
+      out[m.decay_at() + c] = expf(-expf(a_log[c / m.D]) * softplus_f(z[(size_t)t * ldz + c] + dt_bias[c]));
+    return;
+  }
   for (int c = vp * DELTA_V_PIECE + threadIdx.x; c < min(n_v, (vp + 1) * DELTA_V_PIECE); c += blockDim.x)
     out[Nqk + c] = delta_conv_one(proj, ld, carry, conv_w, Nqk + c, Nc, K, pos, p0, r0);
-  if (piece == (int)gridDim.y - 1) {
+  if (vp == v_pieces - 1) {
     const float* row = proj + (size_t)t * ld;
     for (int h = threadIdx.x; h < m.H; h += blockDim.x) {
-      const float b = row[Nc + h], a = row[Nc + m.H + h];
-      out[Nc + h] = 1.0f / (1.0f + expf(-b));
-      out[Nc + m.H + h] = expf(-expf(a_log[h]) * softplus_f(a + dt_bias[h]));
+      out[m.beta_at() + h] = 1.0f / (1.0f + expf(-row[Nc + h]));
+      if (!m.channel) out[m.decay_at() + h] = expf(-expf(a_log[h]) * softplus_f(row[Nc + m.H + h] + dt_bias[h]));
     }
   }
 }
@@ -143,8 +157,9 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
   const int cols = blockDim.x;                               // Dv rounded up to whole warps
   const int j = threadIdx.x;
   const bool live = j < Dv;
-  float* kq = sm;                                            // [2][2*D]: k then q of a token
-  float* S_s = sm + 4 * D;                                   // [D][cols] (DREG == 0 only)
+  const int per = (m.channel ? 3 : 2) * D;
+  float* kq = sm;                                            // [2][2*D]: k then q of a token (then its decays, if per channel)
+  float* S_s = sm + 2 * per;                                 // [D][cols] (DREG == 0 only)
   const int kh = h / (m.H / m.Hk);
   float* S_g = state + (size_t)slot * m.state_floats() + (size_t)h * D * Dv;
   float S_r[DREG > 0 ? DREG : 1];
@@ -156,11 +171,11 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
       for (int d = 0; d < D; ++d) S_s[(size_t)d * cols + j] = S_g[(size_t)j * D + d];
     }
   }
-  const int Nc = m.n_conv();
   auto fetch = [&](int i, int buf) {
     const float* row = prep + (size_t)(r0 + i) * ldp;
-    for (int d = threadIdx.x; d < 2 * D; d += blockDim.x)
-      kq[buf * 2 * D + d] = d < D ? row[(size_t)m.Hk * D + (size_t)kh * D + d] : row[(size_t)kh * D + (d - D)];
+    for (int d = threadIdx.x; d < per; d += blockDim.x)
+      kq[buf * per + d] = d < D ? row[(size_t)m.Hk * D + (size_t)kh * D + d]
+                                : (d < 2 * D ? row[(size_t)kh * D + (d - D)] : row[m.decay_at() + (size_t)h * D + (d - 2 * D)]);
   };
   fetch(0, 0);
   for (int i = 0; i < n; ++i) {
@@ -169,10 +184,28 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
     if (!live) continue;
     const float* row = prep + (size_t)(r0 + i) * ldp;
     const float v = row[(size_t)m.n_qk() + (size_t)h * Dv + j];
-    const float beta = row[Nc + h], g = row[Nc + m.H + h];
-    const float* k = kq + (i & 1) * 2 * D;
+    const float beta = row[m.beta_at() + h];
+    const float* k = kq + (i & 1) * per;
     const float* q = k + D;
     float sk = 0.f;
+    if (m.channel) {
+      const float* gd = q + D;
+      for (int d = 0; d < D; ++d) {
+        const float s = gd[d] * S_s[(size_t)d * cols + j];
+        S_s[(size_t)d * cols + j] = s;
+        sk = fmaf(s, k[d], sk);
+      }
+      const float u = beta * (v - sk);
+      float o = 0.f;
+      for (int d = 0; d < D; ++d) {
+        const float s = fmaf(k[d], u, S_s[(size_t)d * cols + j]);
+        S_s[(size_t)d * cols + j] = s;
+        o = fmaf(s, q[d], o);
+      }
+      o_raw[(size_t)(r0 + i) * ldo + (size_t)h * Dv + j] = o;
+      continue;
+    }
+    const float g = row[m.decay_at() + h];
     if (DREG > 0) {
 #pragma unroll
       for (int d = 0; d < DREG; ++d) sk = fmaf(S_r[d], k[d], sk);
@@ -228,7 +261,7 @@ __device__ __forceinline__ void cp_async16_ca(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 
-template <int D>
+template <int D, bool CH>
 __global__ void __launch_bounds__(256)
 delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, float* __restrict__ state,
                              const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_slot,
@@ -259,20 +292,22 @@ delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims
     S_r[i][2] = make_float2(c0.z, c1.z);
     S_r[i][3] = make_float2(c0.w, c1.w);
   }
-  const int Nc = m.n_conv();
-  // ring entry: [k (D) | q (D) | v of the slice (CB) | beta, g, 0, 0]; all parts are whole 16-byte pieces
-  const int n16 = (2 * D + CB) / 4, pitch = 2 * D + CB + 4;
+  // ring entry: [k (D) | q (D) | v of the slice (CB) | beta, g, 0, 0], or, with a decay per channel,
+  // [k (D) | q (D) | v (CB) | g (D) | beta, 0, 0, 0]; all parts are whole 16-byte pieces
+  constexpr int NG = CH ? D : 0;
+  const int n16 = (2 * D + CB + NG) / 4, pitch = 2 * D + CB + NG + 4;
   const float* k_src = prep + (size_t)m.Hk * D + (size_t)kh * D;
   const float* q_src = prep + (size_t)kh * D;
   const float* v_src = prep + (size_t)m.n_qk() + (size_t)h * Dv + blockIdx.z * CB;
   auto issue = [&](int i) {
     float* dst = sm + (size_t)(i % DELTA_RING) * pitch;
     const size_t row = (size_t)(r0 + i) * ldp;
-    for (int e = threadIdx.x; e < n16 + 2; e += blockDim.x) {
+    for (int e = threadIdx.x; e < n16 + (CH ? 1 : 2); e += blockDim.x) {
       if (e < D / 4) cp_async16_ca(dst + 4 * e, k_src + row + 4 * e);
       else if (e < D / 2) cp_async16_ca(dst + 4 * e, q_src + row + 4 * (e - D / 4));
-      else if (e < n16) cp_async16_ca(dst + 4 * e, v_src + row + 4 * (e - D / 2));
-      else cp_async4(dst + 4 * n16 + (e - n16), prep + row + (e == n16 ? Nc + h : Nc + m.H + h));
+      else if (e < (2 * D + CB) / 4) cp_async16_ca(dst + 4 * e, v_src + row + 4 * (e - D / 2));
+      else if (CH && e < n16) cp_async16_ca(dst + 4 * e, prep + row + m.decay_at() + h * D + 4 * (e - (2 * D + CB) / 4));
+      else cp_async4(dst + 4 * n16 + (e - n16), prep + row + (e == n16 ? m.beta_at() + h : m.decay_at() + h));
     }
   };
 #pragma unroll
@@ -293,8 +328,18 @@ delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims
       qq[c] = holds ? *reinterpret_cast<const float4*>(in + D + 64 * c + 4 * sub) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const float2 v = *reinterpret_cast<const float2*>(in + 2 * D + 2 * cg);
-    const float beta = in[2 * D + CB], g = in[2 * D + CB + 1];
+    const float beta = in[4 * n16], g = CH ? 1.0f : in[4 * n16 + 1];
     float2 sk = make_float2(0.f, 0.f), sk2 = make_float2(0.f, 0.f);
+    if (CH) {                                                // the decay of every row, before anything reads the state
+#pragma unroll
+      for (int c = 0; c < NI; ++c) {
+        const float4 gg = holds ? *reinterpret_cast<const float4*>(in + 2 * D + CB + 64 * c + 4 * sub) : make_float4(0.f, 0.f, 0.f, 0.f);
+        S_r[c][0].x *= gg.x; S_r[c][0].y *= gg.x;
+        S_r[c][1].x *= gg.y; S_r[c][1].y *= gg.y;
+        S_r[c][2].x *= gg.z; S_r[c][2].y *= gg.z;
+        S_r[c][3].x *= gg.w; S_r[c][3].y *= gg.w;
+      }
+    }
 #pragma unroll
     for (int c = 0; c < NI; ++c) {
       sk.x = fmaf(S_r[c][0].x, kk[c].x, sk.x);
@@ -313,7 +358,7 @@ delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims
       sk.x += __shfl_xor_sync(0xffffffffu, sk.x, o);
       sk.y += __shfl_xor_sync(0xffffffffu, sk.y, o);
     }
-    const float ux = beta * (v.x - g * sk.x), uy = beta * (v.y - g * sk.y);
+    const float ux = beta * (v.x - (CH ? sk.x : g * sk.x)), uy = beta * (v.y - (CH ? sk.y : g * sk.y));
     float2 o2 = make_float2(0.f, 0.f), o3 = make_float2(0.f, 0.f);
 #pragma unroll
     for (int c = 0; c < NI; ++c) {
@@ -322,8 +367,8 @@ delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float2 s = S_r[c][e];
-        s.x = fmaf(ke[e], ux, g * s.x);
-        s.y = fmaf(ke[e], uy, g * s.y);
+        s.x = fmaf(ke[e], ux, CH ? s.x : g * s.x);
+        s.y = fmaf(ke[e], uy, CH ? s.y : g * s.y);
         S_r[c][e] = s;
         if (e & 1) {
           o3.x = fmaf(s.x, qe[e], o3.x);
@@ -353,13 +398,13 @@ delta_recurrence_quad_kernel(const float* __restrict__ prep, long ldp, DeltaDims
   }
 }
 
-template <int D>
+template <int D, bool CH>
 int launch_delta_recurrence_quad(const float* prep, long ldp, DeltaDims m, float* state, const int32_t* seq_q_start,
                                  const int32_t* seq_slot, float* o_raw, long ldo, int n_seqs, int write_state,
                                  cudaStream_t stream) {
   const int CB = m.Dv % 32 == 0 ? 32 : 16;                   // columns per block
-  const size_t smem = (size_t)DELTA_RING * (2 * D + CB + 4) * sizeof(float);
-  return launch_pdl(PDL_ATTENTION, delta_recurrence_quad_kernel<D>, dim3(m.H, n_seqs, m.Dv / CB), dim3(8 * CB), smem, stream, prep,
+  const size_t smem = (size_t)DELTA_RING * ((CH ? 3 : 2) * D + CB + 4) * sizeof(float);
+  return launch_pdl(PDL_ATTENTION, delta_recurrence_quad_kernel<D, CH>, dim3(m.H, n_seqs, m.Dv / CB), dim3(8 * CB), smem, stream, prep,
                     ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, write_state);
 }
 
@@ -422,7 +467,7 @@ int launch_delta_recurrence(const float* prep, long ldp, DeltaDims m, float* sta
                             const int32_t* seq_slot, float* o_raw, long ldo, int n_seqs, int write_state,
                             cudaStream_t stream) {
   const int cols = (m.Dv + 31) / 32 * 32;
-  const size_t smem = ((size_t)4 * m.D + (DREG > 0 ? 0 : (size_t)m.D * cols)) * sizeof(float);
+  const size_t smem = ((size_t)(m.channel ? 6 : 4) * m.D + (DREG > 0 ? 0 : (size_t)m.D * cols)) * sizeof(float);
   static PerDevice<size_t> allowed;
   if (smem > 48 * 1024 && allowed.here() < smem) {
     if (cudaFuncSetAttribute(delta_recurrence_kernel<DREG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
@@ -445,17 +490,19 @@ LLMI_EXPORT long llmi_delta_state_floats(int H, int Hk, int D, int Dv, int taps)
   return DeltaDims{H, Hk, D, Dv, taps}.state_floats();
 }
 
+// z (fp32 [n_tokens, ldz], or null): the decay is one per key channel, made from z and dt_bias [H*D].
 LLMI_EXPORT int llmi_delta_prepare(const float* proj, long ld, int H, int Hk, int D, int Dv, int taps, const float* conv_w,
                                    const float* a_log, const float* dt_bias, const float* state, const int32_t* tok_seq,
                                    const int32_t* tok_pos, const int32_t* seq_q_start, const int32_t* seq_slot, float* prep,
-                                   long ldp, int n_tokens, cudaStream_t stream) {
-  const DeltaDims m{H, Hk, D, Dv, taps};
+                                   long ldp, int n_tokens, const float* z, long ldz, cudaStream_t stream) {
+  const DeltaDims m{H, Hk, D, Dv, taps, z != nullptr};
   if (n_tokens <= 0 || !delta_dims_ok(m)) return LLMI_ERR_BAD_SIZE;
-  const int pieces = 2 * m.Hk + (m.H * m.Dv + DELTA_V_PIECE - 1) / DELTA_V_PIECE;
+  const int pieces = 2 * m.Hk + (m.H * m.Dv + DELTA_V_PIECE - 1) / DELTA_V_PIECE +
+                     (m.channel ? (m.H * m.D + DELTA_V_PIECE - 1) / DELTA_V_PIECE : 0);
   if (pieces > 65535) return LLMI_ERR_BAD_SIZE;
   const int threads = m.D >= 256 ? 256 : (m.D > 64 ? 128 : 64);
   return launch_pdl(PDL_SMALL, delta_prepare_kernel, dim3(n_tokens, pieces), dim3(threads), 0, stream, proj, ld, m, conv_w, a_log,
-                    dt_bias, state, tok_seq, tok_pos, seq_q_start, seq_slot, prep, ldp);
+                    dt_bias, state, tok_seq, tok_pos, seq_q_start, seq_slot, prep, ldp, z, ldz);
 }
 
 LLMI_EXPORT int llmi_delta_conv_carry(const float* proj, long ld, int H, int Hk, int D, int Dv, int taps, float* state,
@@ -470,17 +517,21 @@ LLMI_EXPORT int llmi_delta_conv_carry(const float* proj, long ld, int H, int Hk,
 
 LLMI_EXPORT int llmi_delta_recurrence(const float* prep, long ldp, int H, int Hk, int D, int Dv, int taps, float* state,
                                       const int32_t* seq_q_start, const int32_t* seq_slot, float* o_raw, long ldo, int n_seqs,
-                                      int write_state, cudaStream_t stream) {
-  const DeltaDims m{H, Hk, D, Dv, taps};
+                                      int write_state, int channel, cudaStream_t stream) {
+  const DeltaDims m{H, Hk, D, Dv, taps, channel != 0};
   if (n_seqs <= 0 || n_seqs > 65535 || !delta_dims_ok(m)) return LLMI_ERR_BAD_SIZE;
   // (16-byte accesses: state rows, o rows and the ring's v entries must be 16-byte aligned)
   if (Dv % 16 == 0 && ldo % 4 == 0 && ldp % 4 == 0 && !((uintptr_t)state & 15) && !((uintptr_t)o_raw & 15) &&
       !((uintptr_t)prep & 15) && DeltaDims{H, Hk, D, Dv, taps}.state_floats() % 4 == 0) {
-    if (D == 32) return launch_delta_recurrence_quad<32>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream);
-    if (D == 64) return launch_delta_recurrence_quad<64>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream);
-    if (D == 128) return launch_delta_recurrence_quad<128>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream);
+#define LLMI_QUAD(DD)                                                                                                                    \
+  return m.channel ? launch_delta_recurrence_quad<DD, true>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream) \
+                   : launch_delta_recurrence_quad<DD, false>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream)
+    if (D == 32) LLMI_QUAD(32);
+    if (D == 64) LLMI_QUAD(64);
+    if (D == 128) LLMI_QUAD(128);
+#undef LLMI_QUAD
   }
-  if ((size_t)D * ((Dv + 31) / 32 * 32) * 4 + 16 * (size_t)D > 200 * 1024) return LLMI_ERR_BAD_SIZE;
+  if ((size_t)D * ((Dv + 31) / 32 * 32) * 4 + 24 * (size_t)D > 200 * 1024) return LLMI_ERR_BAD_SIZE;
   return launch_delta_recurrence<0>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream);
 }
 

@@ -63,6 +63,8 @@ struct SkinnyParams {
   int in_tiles;
   float in_eps;
   int act;                    // the gate's activation in mode SK_SWIGLU (see gated_value); in mode SK_STORE 2: relu(v)^2 is stored
+  const float* oscale;        // [m_out] or null: the value with its bias is multiplied by it (not in mode SK_SWIGLU)
+  GateConstants gate;
 };
 
 // One copy fetches [4 k slices][rows][64 k]: the matrix is seen as a 3-D tensor (k within a slice, row, slice).
@@ -243,10 +245,10 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
           float v = 0.f;
 #pragma unroll
           for (int w = 0; w < SK_CONSUMERS; ++w) v += s_part[w][ln][n * 4 + e];
-          gu[h] = v * sc;
+          gu[h] = v * sc + (p.bias ? p.bias[m0 + row] : 0.f);
         }
         ((__nv_bfloat16*)p.out)[(size_t)tok * p.ldo + (m0 >> 1) + f] =
-            __float2bfloat16_rn(gated_value(gu[0], gu[1], p.act));
+            __float2bfloat16_rn(gated_value(gu[0], gu[1], p.act, p.gate));
       }
     } else {
       // NPAD * 16 is a multiple of the 128 consumer threads: every thread makes the same number of rounds, and
@@ -265,6 +267,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         float xn = 0.f;
         if (live) {
           if (p.bias) v += p.bias[m];
+          if (p.oscale) v *= p.oscale[m];
           const size_t o = (size_t)tok * p.ldo + m;
           if (p.mode == SK_STORE) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(stored_value(v, p.act));
           else if (p.mode == SK_STORE_F32) ((float*)p.out)[o] = v;
@@ -343,17 +346,17 @@ LLMI_EXPORT int llmi_gemm_skinny_max_tokens() { return 64; }
 // modes as llmi_gemm_tc (0 store, 1 fp32 store, 2 fp32 add, 3 gated with alternating gate/up rows).
 // emit_w/emit_h/emit_ss (mode 2 only, or all null): also write h = bf16(emit_w * y_new) and the per-tile sums of
 // y_new^2, emit_ss[ceil(m_out/16), 64].  in_ss/in_tiles/in_eps (or null): x is such an h; the accumulators are
-// multiplied by 1/sqrt(sum of the tiles' sums / k + in_eps) before the bias.
+// multiplied by 1/sqrt(sum of the tiles' sums / k + in_eps) before the bias.  oscale, gate_alpha, gate_limit: as llmi_gemm_tc.
 LLMI_EXPORT int llmi_gemm_skinny(const void* x, long ldx, const void* w, long ldw, const float* bias, void* y, long ldy,
                                  int n_tok, int m_out, int k, int mode, const float* emit_w, void* emit_h, long emit_ldh,
                                  float* emit_ss, const float* in_ss, int in_tiles, float in_eps, int* error_flag,
-                                 cudaStream_t stream) {
+                                 const float* oscale, float gate_alpha, float gate_limit, cudaStream_t stream) {
   if (n_tok <= 0 || n_tok > 64 || m_out <= 0 || k <= 0) return LLMI_ERR_BAD_SIZE;
-  if (mode < 0 || mode > OUT_GELU_REQUEST) return LLMI_ERR_UNSUPPORTED;
-  const int act = mode == OUT_GEGLU_REQUEST ? 1 : store_act_of(mode);
-  if (mode == OUT_GEGLU_REQUEST) mode = SK_SWIGLU;
+  if (mode < 0 || mode > OUT_BOUNDED_REQUEST) return LLMI_ERR_UNSUPPORTED;
+  const int act = mode == OUT_GEGLU_REQUEST ? 1 : (mode == OUT_BOUNDED_REQUEST ? ACT_BOUNDED : store_act_of(mode));
+  if (mode == OUT_GEGLU_REQUEST || mode == OUT_BOUNDED_REQUEST) mode = SK_SWIGLU;
   if (mode == OUT_RELU2_REQUEST || mode == OUT_GELU_REQUEST) mode = SK_STORE;
-  if (mode == SK_SWIGLU && ((m_out & 1) || bias)) return LLMI_ERR_UNSUPPORTED;
+  if (mode == SK_SWIGLU && ((m_out & 1) || oscale)) return LLMI_ERR_UNSUPPORTED;
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15) || (ldx & 7) || (ldw & 7)) return LLMI_ERR_ALIGN;
   if (k % 64) return LLMI_ERR_UNSUPPORTED;   // the 3-D view of the matrices needs whole 64-wide k slices
   if (emit_w && (mode != SK_ADD_F32 || !emit_h || !emit_ss)) return LLMI_ERR_UNSUPPORTED;
@@ -365,7 +368,7 @@ LLMI_EXPORT int llmi_gemm_skinny(const void* x, long ldx, const void* w, long ld
   rc = sk_make_map(&mx, x, n_tok, k, ldx, n_tok);
   if (rc != LLMI_OK) return rc;
   SkinnyParams p{m_out, n_tok, k, y, ldy, bias, mode, error_flag, n_tok, emit_w, (__nv_bfloat16*)emit_h, emit_ldh, emit_ss,
-                 in_ss, in_tiles, in_eps, act};
+                 in_ss, in_tiles, in_eps, act, oscale, GateConstants{gate_alpha, gate_limit}};
   const int m_tiles = (m_out + SK_ROWS - 1) / SK_ROWS;
   if (nt == 1) return launch_skinny<1>(mw, mx, p, m_tiles, stream);
   if (nt == 2) return launch_skinny<2>(mw, mx, p, m_tiles, stream);

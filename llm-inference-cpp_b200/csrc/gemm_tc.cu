@@ -200,7 +200,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         // that their round trip to L2 overlaps the chunk before (and, for the first chunk, the MMAs).
         const int nch = (min(BN, p.n_tok - n0) + 15) / 16;
         const bool row_ok = m < p.m_out;
-        const float bias = (p.bias && row_ok) ? p.bias[m] : 0.f;
+        const float bias = (p.bias && row_ok) ? p.bias[m] : 0.f, os = (p.oscale && row_ok) ? p.oscale[m] : 1.f;
         float* o = (float*)p.out + (size_t)n0 * p.ldo + m;
         float nxt[16];
 #pragma unroll
@@ -224,7 +224,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           }
 #pragma unroll
           for (int c = 0; c < 16; ++c)
-            if (row_ok && n0 + ci * 16 + c < p.n_tok) o[(size_t)(ci * 16 + c) * p.ldo] = cur[c] + (v[c] + bias);
+            if (row_ok && n0 + ci * 16 + c < p.n_tok) o[(size_t)(ci * 16 + c) * p.ldo] = cur[c] + (v[c] + bias) * os;
         }
         continue;
       }
@@ -439,7 +439,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
         // (gated, the stores of the threads cost 7 to 10 us a product that the next tile's MMAs did not hide; it is
         // not hidden at all when a pair has one tile only: the o and down projections of a 2,048-token prompt).
         // Rows and tokens past the ends of `out` are clipped by the copy.
-        const float bias = (p.bias && m < p.m_out) ? p.bias[m] : 0.f;
+        const float bias = (p.bias && m < p.m_out) ? p.bias[m] : 0.f, os = (p.oscale && m < p.m_out) ? p.oscale[m] : 1.f;
         const int row_in_cta = quad * 32 + lane;
         for (int ci = 0; ci < nch; ++ci) {
           float v[16];
@@ -461,6 +461,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             // rows alternate gate and up (src/model/transformer.cpp:290; src/model/kernels.cpp:148): the even lane finishes
             // tokens 0..7 of feature row / 2, the odd lane tokens 8..15
             const bool is_gate = (row_in_cta & 1) == 0;
+            if (p.bias) {                                    // a row's own bias, before the exchange
+#pragma unroll
+              for (int c = 0; c < 16; ++c) v[c] += bias;
+            }
             float g[8], u[8];
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
@@ -470,15 +474,15 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             }
             __nv_bfloat16* o = (__nv_bfloat16*)bufp + (is_gate ? 0 : 8) * (TC_BM / 2) + (row_in_cta >> 1);
 #pragma unroll
-            for (int c = 0; c < 8; ++c) o[c * (TC_BM / 2)] = __float2bfloat16_rn(gated_value(g[c], u[c], p.act));
+            for (int c = 0; c < 8; ++c) o[c * (TC_BM / 2)] = __float2bfloat16_rn(gated_value(g[c], u[c], p.act, p.gate));
           } else if (p.mode == OUT_STORE) {
             __nv_bfloat16* o = (__nv_bfloat16*)bufp + row_in_cta;
 #pragma unroll
-            for (int c = 0; c < 16; ++c) o[c * TC_BM] = __float2bfloat16_rn(stored_value(v[c] + bias, p.act));
+            for (int c = 0; c < 16; ++c) o[c * TC_BM] = __float2bfloat16_rn(stored_value((v[c] + bias) * os, p.act));
           } else {
             float* o = (float*)bufp + row_in_cta;
 #pragma unroll
-            for (int c = 0; c < 16; ++c) o[c * TC_BM] = v[c] + bias;
+            for (int c = 0; c < 16; ++c) o[c * TC_BM] = (v[c] + bias) * os;
           }
           asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
           asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -703,23 +707,28 @@ __device__ __forceinline__ void wide_way_out(const TcParams& p, const CUtensorMa
     // rows alternate gate and up (src/model/transformer.cpp:290; src/model/kernels.cpp:148): the even lane takes the
     // odd lane's up and finishes feature row / 2
     __nv_bfloat16* o = (__nv_bfloat16*)stg + (size_t)(cg * CPT) * (RP / 2) + (row >> 1);
+    if (p.bias) {                                            // a row's own bias, before the exchange
+      const float b = m < p.m_out ? p.bias[m] : 0.f;
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) v[c] += b;
+    }
     float up[CPT];
 #pragma unroll
     for (int c = 0; c < CPT; ++c) up[c] = __shfl_down_sync(0xffffffffu, v[c], 1);
     if (!(row & 1)) {
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) o[c * (RP / 2)] = __float2bfloat16_rn(gated_value(v[c], up[c], p.act));
+      for (int c = 0; c < CPT; ++c) o[c * (RP / 2)] = __float2bfloat16_rn(gated_value(v[c], up[c], p.act, p.gate));
     }
   } else {
-    const float b = (p.bias && m < p.m_out) ? p.bias[m] : 0.f;
+    const float b = (p.bias && m < p.m_out) ? p.bias[m] : 0.f, os = (p.oscale && m < p.m_out) ? p.oscale[m] : 1.f;
     if (p.mode == OUT_STORE) {
       __nv_bfloat16* o = (__nv_bfloat16*)stg + (size_t)(cg * CPT) * RP + row;
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) o[c * RP] = __float2bfloat16_rn(stored_value(v[c] + b, p.act));
+      for (int c = 0; c < CPT; ++c) o[c * RP] = __float2bfloat16_rn(stored_value((v[c] + b) * os, p.act));
     } else {
       float* o = (float*)stg + (size_t)(cg * CPT) * RP + row;
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) o[c * RP] = v[c] + b;
+      for (int c = 0; c < CPT; ++c) o[c * RP] = (v[c] + b) * os;
     }
   }
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the staging tile is read by the async proxy
@@ -1094,17 +1103,20 @@ LLMI_EXPORT long llmi_gemm_tc_workspace(int n_tok, int m_out, int k, int* n_tick
 
 // y[n_tok, m_out] (mode) = x[n_tok, k] · w[m_out, k]ᵀ + bias; bf16 inputs; pitches in elements.
 // mode 3 (gated): w's rows alternate gate and up rows of a feed-forward, y is [n_tok, m_out / 2] bf16 and
-// receives silu(gate) * up.
+// receives silu(gate) * up (mode 4: the tanh form of GELU; mode 7: the bounded gate with the constants gate_alpha and
+// gate_limit); a bias is then [m_out] in the rows' order.  oscale ([m_out] or null; ungated modes): y takes (x · wᵀ + bias) * oscale.
 // Requirements (else LLMI_ERR_ALIGN): x, w 16-byte aligned; ldx, ldw multiples of 8 elements.
 LLMI_EXPORT int llmi_gemm_tc(const void* x, long ldx, const void* w, long ldw, const float* bias, void* y, long ldy,
                              int n_tok, int m_out, int k, int mode, float* workspace, long workspace_bytes,
-                             int* tickets, int n_tickets, int* error_flag, cudaStream_t stream) {
+                             int* tickets, int n_tickets, int* error_flag, const float* oscale, float gate_alpha,
+                             float gate_limit, cudaStream_t stream) {
   if (n_tok <= 0 || m_out <= 0 || k <= 0) return LLMI_ERR_BAD_SIZE;
-  if (mode < 0 || mode > OUT_GELU_REQUEST) return LLMI_ERR_UNSUPPORTED;
-  const int act = mode == OUT_GEGLU_REQUEST ? 1 : store_act_of(mode);
-  if (mode == OUT_GEGLU_REQUEST) mode = OUT_SWIGLU;
+  if (mode < 0 || mode > OUT_BOUNDED_REQUEST) return LLMI_ERR_UNSUPPORTED;
+  const int act = mode == OUT_GEGLU_REQUEST ? 1 : (mode == OUT_BOUNDED_REQUEST ? ACT_BOUNDED : store_act_of(mode));
+  const GateConstants gate{gate_alpha, gate_limit};
+  if (mode == OUT_GEGLU_REQUEST || mode == OUT_BOUNDED_REQUEST) mode = OUT_SWIGLU;
   if (mode == OUT_RELU2_REQUEST || mode == OUT_GELU_REQUEST) mode = OUT_STORE;
-  if (mode == OUT_SWIGLU && ((m_out & 1) || bias)) return LLMI_ERR_UNSUPPORTED;
+  if (mode == OUT_SWIGLU && ((m_out & 1) || oscale)) return LLMI_ERR_UNSUPPORTED;
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15) || (ldx & 7) || (ldw & 7)) return LLMI_ERR_ALIGN;
   const int bn = tc_bn(n_tok, m_out);
   int need_tickets = 0;
@@ -1120,7 +1132,7 @@ LLMI_EXPORT int llmi_gemm_tc(const void* x, long ldx, const void* w, long ldw, c
     if (rc != LLMI_OK) return rc;
     rc = boxed3d ? make_map_3d(&mx, x, n_tok, k, ldx, bn, 2) : make_map(&mx, x, n_tok, k, ldx, bn);
     if (rc != LLMI_OK) return rc;
-    TcParams pk{m_out, n_tok, k, y, ldy, bias, mode, 1, nullptr, nullptr, error_flag, act};
+    TcParams pk{m_out, n_tok, k, y, ldy, bias, mode, 1, nullptr, nullptr, error_flag, act, oscale, gate};
     const int m_tiles = (m_out + TC_BM - 1) / TC_BM, n_tiles = (n_tok + bn - 1) / bn;
     // the way out by TMA: a CTA of a cluster of W stores [bn tokens][128 / W rows] (gated: half as many features)
     CUtensorMap mo = mw;
@@ -1155,13 +1167,13 @@ LLMI_EXPORT int llmi_gemm_tc(const void* x, long ldx, const void* w, long ldw, c
       const int pbn = pair_token_tile(n_tok, m_out);
       rc = make_map(&mx, x, n_tok, k, ldx, pbn / 2);
       if (rc != LLMI_OK) return rc;
-      TcParams pp{m_out, n_tok, k, y, ldy, bias, mode, 1, workspace, tickets, error_flag, act};
+      TcParams pp{m_out, n_tok, k, y, ldy, bias, mode, 1, workspace, tickets, error_flag, act, oscale, gate};
       return launch_tc_pair(mw, mx, mo, pp, (m_out + 255) / 256, (n_tok + pbn - 1) / pbn, pbn, out_rc == LLMI_OK, stream);
     }
   }
   rc = make_map(&mx, x, n_tok, k, ldx, bn);
   if (rc != LLMI_OK) return rc;
-  TcParams p{m_out, n_tok, k, y, ldy, bias, mode, splits, workspace, tickets, error_flag, act};
+  TcParams p{m_out, n_tok, k, y, ldy, bias, mode, splits, workspace, tickets, error_flag, act, oscale, gate};
   const int m_tiles = (m_out + TC_BM - 1) / TC_BM, n_tiles = (n_tok + bn - 1) / bn;
   if ((long)m_tiles * n_tiles * splits > 0x7fffffffL) return LLMI_ERR_BAD_SIZE;
   switch (bn) {

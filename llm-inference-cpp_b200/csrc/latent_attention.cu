@@ -13,7 +13,8 @@
 //   llmi_attention_latent   scores, softmax and context of every (token, head), any sizes, fp32 arithmetic; serves
 //                           prompts and single tokens, both types; optionally over a window of the last positions only
 // Rotation: pairs turned by the angle float(pos) * inv_freq[i], computed in fp32 with sincosf — neighbours (2i, 2i+1)
-// (`pairing` 1) or entries (i, i + rot_dims/2) (`pairing` 0); entries beyond rot_dims pass unchanged.
+// (`pairing` 1) or entries (i, i + rot_dims/2) (`pairing` 0), cos and sin both times `amplitude`; entries beyond rot_dims
+// pass unchanged.
 #include <math.h>
 
 #include "common.cuh"
@@ -30,12 +31,14 @@ __device__ __forceinline__ void pair_places(int i, int rot_dims, int pairing, in
 // R entries of src, the first rot_dims of them turned by the position, into dst; thread `me` of `n`.
 template <typename T>
 __device__ __forceinline__ void rotate_part(const float* __restrict__ src, T* __restrict__ dst, int R, const float* __restrict__ inv_freq,
-                                            int rot_dims, int pairing, int pos, int me, int n) {
+                                            int rot_dims, int pairing, float amplitude, int pos, int me, int n) {
   for (int i = me; i < rot_dims / 2; i += n) {
     int a, b;
     pair_places(i, rot_dims, pairing, a, b);
     float s, co;
     sincosf((float)pos * inv_freq[i], &s, &co);
+    s *= amplitude;
+    co *= amplitude;
     dst[a] = from_f32<T>(rot_lo(src[a], src[b], co, s));
     dst[b] = from_f32<T>(rot_hi(src[a], src[b], co, s));
   }
@@ -50,7 +53,7 @@ __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const float* __restrict__ down, long ld, int Q, int C, int R, const float* __restrict__ wq,
                       const float* __restrict__ wc, float eps, const float* __restrict__ inv_freq, int rot_dims,
                       const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos, PagedKV kv,
-                      T* __restrict__ cache, T* __restrict__ cq, int write_kv, int pairing) {
+                      T* __restrict__ cache, T* __restrict__ cq, int write_kv, int pairing, float amplitude) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -77,7 +80,7 @@ latent_prepare_kernel(const float* __restrict__ down, long ld, int Q, int C, int
   T* dst = cache + kv_row_offset(kv, seq, pos, 0);
   for (int i = threadIdx.x; i < C; i += blockDim.x) dst[i] = from_f32<T>(wc[i] * (c[i] * sc));
   const float* r = c + C;
-  rotate_part<T>(r, dst + C, R, inv_freq, rot_dims, pairing, pos, threadIdx.x, blockDim.x);
+  rotate_part<T>(r, dst + C, R, inv_freq, rot_dims, pairing, amplitude, pos, threadIdx.x, blockDim.x);
 }
 
 // The same for a layer whose queries come straight from its input.  proj: fp32 [T, ld]: [ q: H * (D + R) | c: C | r: R ].
@@ -90,7 +93,7 @@ __global__ void __launch_bounds__(LP_WARPS * 32)
 latent_prepare_direct_kernel(const float* __restrict__ proj, long ld, int H, int D, int C, int R, const float* __restrict__ wc,
                              float eps, const float* __restrict__ inv_freq, int rot_dims, int pairing,
                              const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos, PagedKV kv,
-                             T* __restrict__ cache, T* __restrict__ qn, T* __restrict__ qa, long ldqa, int n_tokens, int write_kv) {
+                             T* __restrict__ cache, T* __restrict__ qn, T* __restrict__ qa, long ldqa, int n_tokens, int write_kv, float amplitude) {
   pdl_launch_dependents();
   pdl_wait();
   const long item = (long)blockIdx.x * LP_WARPS + (threadIdx.x >> 5);
@@ -109,7 +112,7 @@ latent_prepare_direct_kernel(const float* __restrict__ proj, long ld, int H, int
       return;
     }
     for (int i = lane; i < D; i += 32) plain[i] = from_f32<T>(src[i]);
-    rotate_part<T>(src + D, rot, R, inv_freq, rot_dims, pairing, tok_pos[t], lane, 32);
+    rotate_part<T>(src + D, rot, R, inv_freq, rot_dims, pairing, amplitude, tok_pos[t], lane, 32);
     return;
   }
   if (seq < 0 || !write_kv) return;
@@ -120,7 +123,7 @@ latent_prepare_direct_kernel(const float* __restrict__ proj, long ld, int H, int
   const int pos = tok_pos[t];
   T* dst = cache + kv_row_offset(kv, seq, pos, 0);
   for (int i = lane; i < C; i += 32) dst[i] = from_f32<T>(wc[i] * (c[i] * sc));
-  rotate_part<T>(c + C, dst + C, R, inv_freq, rot_dims, pairing, pos, lane, 32);
+  rotate_part<T>(c + C, dst + C, R, inv_freq, rot_dims, pairing, amplitude, pos, lane, 32);
 }
 
 // q (type T) [T, H, D + R] holds every head's plain part and its part to rotate; qa [T, H, C + R] receives the
@@ -129,7 +132,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 latent_q_rotate_kernel(const T* __restrict__ q, long ldq, int D, T* __restrict__ qa, long ldqa, int C, int R, int H,
                        const float* __restrict__ inv_freq, int rot_dims, const int32_t* __restrict__ tok_seq,
-                       const int32_t* __restrict__ tok_pos, int n_tokens, int pairing) {
+                       const int32_t* __restrict__ tok_pos, int n_tokens, int pairing, float amplitude) {
   pdl_launch_dependents();
   pdl_wait();
   const int half = rot_dims / 2 + (R - rot_dims + 1) / 2;      // the pairs that turn, then the rest two by two
@@ -150,6 +153,8 @@ latent_q_rotate_kernel(const T* __restrict__ q, long ldq, int D, T* __restrict__
     if (i < rot_dims / 2) {
       float s, co;
       sincosf((float)tok_pos[t] * inv_freq[i], &s, &co);
+      s *= amplitude;
+      co *= amplitude;
       const float u = to_f32(src[a]), v = to_f32(src[b]);
       dst[a] = from_f32<T>(rot_lo(u, v, co, s));
       dst[b] = from_f32<T>(rot_hi(u, v, co, s));
@@ -288,15 +293,15 @@ LLMI_EXPORT int llmi_latent_prepare(int dtype, const float* down, long ld, int Q
                                     const float* wc, float eps, const float* inv_freq, int rot_dims,
                                     const int32_t* tok_seq, const int32_t* tok_pos, const int32_t* seq_pages,
                                     int pages_stride, int page_size, void* cache, void* cq, int n_tokens, int write_kv,
-                                    int pairing, cudaStream_t stream) {
+                                    int pairing, float amplitude, cudaStream_t stream) {
   if (n_tokens <= 0 || Q <= 0 || C <= 0 || R < 0 || rot_dims < 0 || rot_dims > R || (rot_dims & 1)) return LLMI_ERR_BAD_SIZE;
   PagedKV kv{seq_pages, pages_stride, page_size, 1, C + R};
   if (dtype == LLMI_DTYPE_F32)
     return launch_pdl(PDL_ROPE, latent_prepare_kernel<float>, n_tokens, 128, 0, stream, down, ld, Q, C, R, wq, wc, eps, inv_freq,
-                      rot_dims, tok_seq, tok_pos, kv, (float*)cache, (float*)cq, write_kv, pairing);
+                      rot_dims, tok_seq, tok_pos, kv, (float*)cache, (float*)cq, write_kv, pairing, amplitude);
   if (dtype == LLMI_DTYPE_BF16)
     return launch_pdl(PDL_ROPE, latent_prepare_kernel<__nv_bfloat16>, n_tokens, 128, 0, stream, down, ld, Q, C, R, wq, wc, eps,
-                      inv_freq, rot_dims, tok_seq, tok_pos, kv, (__nv_bfloat16*)cache, (__nv_bfloat16*)cq, write_kv, pairing);
+                      inv_freq, rot_dims, tok_seq, tok_pos, kv, (__nv_bfloat16*)cache, (__nv_bfloat16*)cq, write_kv, pairing, amplitude);
   return LLMI_ERR_BAD_DTYPE;
 }
 
@@ -305,7 +310,7 @@ LLMI_EXPORT int llmi_latent_prepare(int dtype, const float* down, long ld, int Q
 LLMI_EXPORT int llmi_latent_prepare_direct(int dtype, const float* proj, long ld, int H, int D, int C, int R, const float* wc,
                                            float eps, const float* inv_freq, int rot_dims, int pairing, const int32_t* tok_seq,
                                            const int32_t* tok_pos, const int32_t* seq_pages, int pages_stride, int page_size,
-                                           void* cache, void* qn, void* qa, long ldqa, int n_tokens, int write_kv,
+                                           void* cache, void* qn, void* qa, long ldqa, int n_tokens, int write_kv, float amplitude,
                                            cudaStream_t stream) {
   if (n_tokens <= 0 || H <= 0 || D <= 0 || C <= 0 || R < 0 || rot_dims < 0 || rot_dims > R || (rot_dims & 1) || page_size <= 0)
     return LLMI_ERR_BAD_SIZE;
@@ -315,17 +320,17 @@ LLMI_EXPORT int llmi_latent_prepare_direct(int dtype, const float* proj, long ld
   if (dtype == LLMI_DTYPE_F32)
     return launch_pdl(PDL_ROPE, latent_prepare_direct_kernel<float>, dim3((unsigned)blocks), dim3(LP_WARPS * 32), 0, stream, proj, ld, H, D,
                       C, R, wc, eps, inv_freq, rot_dims, pairing, tok_seq, tok_pos, kv, (float*)cache, (float*)qn, (float*)qa, ldqa,
-                      n_tokens, write_kv);
+                      n_tokens, write_kv, amplitude);
   if (dtype == LLMI_DTYPE_BF16)
     return launch_pdl(PDL_ROPE, latent_prepare_direct_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(LP_WARPS * 32), 0, stream, proj,
                       ld, H, D, C, R, wc, eps, inv_freq, rot_dims, pairing, tok_seq, tok_pos, kv, (__nv_bfloat16*)cache,
-                      (__nv_bfloat16*)qn, (__nv_bfloat16*)qa, ldqa, n_tokens, write_kv);
+                      (__nv_bfloat16*)qn, (__nv_bfloat16*)qa, ldqa, n_tokens, write_kv, amplitude);
   return LLMI_ERR_BAD_DTYPE;
 }
 
 LLMI_EXPORT int llmi_latent_q_rotate(int dtype, const void* q, long ldq, int D, void* qa, long ldqa, int C, int R, int H,
                                      const float* inv_freq, int rot_dims, const int32_t* tok_seq, const int32_t* tok_pos,
-                                     int n_tokens, int pairing, cudaStream_t stream) {
+                                     int n_tokens, int pairing, float amplitude, cudaStream_t stream) {
   if (n_tokens <= 0 || H <= 0 || D < 0 || C <= 0 || R < 0 || rot_dims > R || (rot_dims & 1)) return LLMI_ERR_BAD_SIZE;
   if (R == 0) return LLMI_OK;
   const size_t total = (size_t)n_tokens * H * (rot_dims / 2 + (R - rot_dims + 1) / 2);
@@ -333,10 +338,10 @@ LLMI_EXPORT int llmi_latent_q_rotate(int dtype, const void* q, long ldq, int D, 
   const int blocks = (int)(need < most ? need : most);
   if (dtype == LLMI_DTYPE_F32)
     return launch_pdl(PDL_SMALL, latent_q_rotate_kernel<float>, blocks, 256, 0, stream, (const float*)q, ldq, D, (float*)qa, ldqa, C,
-                      R, H, inv_freq, rot_dims, tok_seq, tok_pos, n_tokens, pairing);
+                      R, H, inv_freq, rot_dims, tok_seq, tok_pos, n_tokens, pairing, amplitude);
   if (dtype == LLMI_DTYPE_BF16)
     return launch_pdl(PDL_SMALL, latent_q_rotate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)q, ldq, D,
-                      (__nv_bfloat16*)qa, ldqa, C, R, H, inv_freq, rot_dims, tok_seq, tok_pos, n_tokens, pairing);
+                      (__nv_bfloat16*)qa, ldqa, C, R, H, inv_freq, rot_dims, tok_seq, tok_pos, n_tokens, pairing, amplitude);
   return LLMI_ERR_BAD_DTYPE;
 }
 

@@ -20,7 +20,7 @@ constexpr int OUT_ADD_F32 = 2;    // y (float) += acc       (residual sum kept i
 template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 linear_simt_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ w, long ldw,
-                   const float* __restrict__ bias, void* __restrict__ yv, long ldy, int M, int N, int K,
+                   const float* __restrict__ bias, const float* __restrict__ oscale, void* __restrict__ yv, long ldy, int M, int N, int K,
                    long bx, long bw, long by) {
   // blockIdx.z numbers the products of a batch (one per head, say): operand b starts bx, bw, by elements further on
   x += (long)blockIdx.z * bx;
@@ -86,6 +86,7 @@ linear_simt_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ w, l
       if (n >= N) continue;
       float v = acc[i][j];
       if (bias) v += bias[n];
+      if (oscale) v *= oscale[n];
       if (MODE == OUT_STORE) {
         ((T*)yv)[(long)m * ldy + n] = from_f32<T>(v);
       } else if (MODE == OUT_STORE_F32) {
@@ -99,19 +100,19 @@ linear_simt_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ w, l
 }
 
 template <typename T>
-int launch_linear_simt(const void* x, long ldx, const void* w, long ldw, const float* bias, void* y, long ldy, int M,
+int launch_linear_simt(const void* x, long ldx, const void* w, long ldw, const float* bias, const float* oscale, void* y, long ldy, int M,
                        int N, int K, int mode, cudaStream_t stream, int batch = 1, long bx = 0, long bw = 0, long by = 0) {
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, batch);
   if (grid.y > 65535 || batch < 1 || batch > 65535) return LLMI_ERR_BAD_SIZE;
   switch (mode) {
     case OUT_STORE:
-      linear_simt_kernel<T, OUT_STORE><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, y, ldy, M, N, K, bx, bw, by);
+      linear_simt_kernel<T, OUT_STORE><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, oscale, y, ldy, M, N, K, bx, bw, by);
       break;
     case OUT_STORE_F32:
-      linear_simt_kernel<T, OUT_STORE_F32><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, y, ldy, M, N, K, bx, bw, by);
+      linear_simt_kernel<T, OUT_STORE_F32><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, oscale, y, ldy, M, N, K, bx, bw, by);
       break;
     case OUT_ADD_F32:
-      linear_simt_kernel<T, OUT_ADD_F32><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, y, ldy, M, N, K, bx, bw, by);
+      linear_simt_kernel<T, OUT_ADD_F32><<<grid, 256, 0, stream>>>((const T*)x, ldx, (const T*)w, ldw, bias, oscale, y, ldy, M, N, K, bx, bw, by);
       break;
     default:
       return LLMI_ERR_UNSUPPORTED;
@@ -123,13 +124,14 @@ int launch_linear_simt(const void* x, long ldx, const void* w, long ldw, const f
 
 using namespace llmi;
 
-// x [M, K] (row pitch ldx), w [N, K] (row pitch ldw), y [M, N] (row pitch ldy), pitches in elements.
-LLMI_EXPORT int llmi_linear_simt(int dtype, const void* x, long ldx, const void* w, long ldw, const float* bias,
+// x [M, K] (row pitch ldx), w [N, K] (row pitch ldw), y [M, N] (row pitch ldy), pitches in elements; y takes
+// (x · wᵀ + bias) * oscale, both [N] or null.
+LLMI_EXPORT int llmi_linear_simt(int dtype, const void* x, long ldx, const void* w, long ldw, const float* bias, const float* oscale,
                                  void* y, long ldy, int M, int N, int K, int mode, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return LLMI_ERR_BAD_SIZE;
-  if (dtype == LLMI_DTYPE_F32) return launch_linear_simt<float>(x, ldx, w, ldw, bias, y, ldy, M, N, K, mode, stream);
+  if (dtype == LLMI_DTYPE_F32) return launch_linear_simt<float>(x, ldx, w, ldw, bias, oscale, y, ldy, M, N, K, mode, stream);
   if (dtype == LLMI_DTYPE_BF16)
-    return launch_linear_simt<__nv_bfloat16>(x, ldx, w, ldw, bias, y, ldy, M, N, K, mode, stream);
+    return launch_linear_simt<__nv_bfloat16>(x, ldx, w, ldw, bias, oscale, y, ldy, M, N, K, mode, stream);
   return LLMI_ERR_BAD_DTYPE;
 }
 
@@ -141,8 +143,8 @@ LLMI_EXPORT int llmi_linear_simt_batched(int dtype, const void* x, long ldx, lon
                                          cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return LLMI_ERR_BAD_SIZE;
   if (dtype == LLMI_DTYPE_F32)
-    return launch_linear_simt<float>(x, ldx, w, ldw, nullptr, y, ldy, M, N, K, mode, stream, batch, bx, bw, by);
+    return launch_linear_simt<float>(x, ldx, w, ldw, nullptr, nullptr, y, ldy, M, N, K, mode, stream, batch, bx, bw, by);
   if (dtype == LLMI_DTYPE_BF16)
-    return launch_linear_simt<__nv_bfloat16>(x, ldx, w, ldw, nullptr, y, ldy, M, N, K, mode, stream, batch, bx, bw, by);
+    return launch_linear_simt<__nv_bfloat16>(x, ldx, w, ldw, nullptr, nullptr, y, ldy, M, N, K, mode, stream, batch, bx, bw, by);
   return LLMI_ERR_BAD_DTYPE;
 }

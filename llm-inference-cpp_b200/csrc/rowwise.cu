@@ -148,21 +148,22 @@ rmsnorm_warp_kernel(const float* __restrict__ x, const float* __restrict__ weigh
 }
 
 // gate_up is [rows, 2*inner]: gate in the first half of a row, up in the second.  ACT 0: silu(g) = g / (1 + exp(-g));
-// ACT 1: the tanh form of GELU, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
-template <int ACT> __device__ __forceinline__ float gate_act(float g) {
-  if (ACT == 0) return g / (1.0f + expf(-g));
-  return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+// ACT 1: the tanh form of GELU, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))); ACT 2: the bounded gate (common.cuh).
+template <int ACT> __device__ __forceinline__ float gate_pair(float g, float u, const GateConstants& c) {
+  if (ACT == 0) return g / (1.0f + expf(-g)) * u;
+  if (ACT == 2) return bounded_gate(g, u, c.alpha, c.limit);
+  return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
 
 template <typename T, int ACT>
-__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inner, size_t total) {
+__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inner, size_t total, GateConstants gc) {
   pdl_launch_dependents();
   pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t r = i / inner, c = i - r * inner;
     const float g = to_f32(gate_up[r * 2 * inner + c]);
     const float u = to_f32(gate_up[r * 2 * inner + inner + c]);
-    out[i] = from_f32<T>(gate_act<ACT>(g) * u);
+    out[i] = from_f32<T>(gate_pair<ACT>(g, u, gc));
   }
 }
 
@@ -280,24 +281,26 @@ LLMI_EXPORT int llmi_copy_to_host(void* dst, const void* src, long bytes, cudaSt
   return cudaStreamSynchronize(stream) == cudaSuccess ? LLMI_OK : LLMI_ERR_LAUNCH;
 }
 
-LLMI_EXPORT int llmi_swiglu(int dtype, const void* gate_up, void* out, int n_rows, int inner, int act, cudaStream_t stream) {
+template <typename T>
+static int launch_swiglu(const void* gate_up, void* out, int inner, int act, size_t total, GateConstants gc, int blocks, int threads,
+                         cudaStream_t stream) {
+  auto kernel = act == 0 ? swiglu_kernel<T, 0> : (act == 1 ? swiglu_kernel<T, 1> : swiglu_kernel<T, 2>);
+  return launch_pdl(PDL_SMALL, kernel, blocks, threads, 0, stream, (const T*)gate_up, (T*)out, inner, total, gc);
+}
+
+// act: 0 silu, 1 the tanh form of GELU, 2 the bounded gate with its two constants.
+LLMI_EXPORT int llmi_swiglu(int dtype, const void* gate_up, void* out, int n_rows, int inner, int act, float alpha, float limit,
+                            cudaStream_t stream) {
   if (n_rows <= 0 || inner <= 0) return LLMI_ERR_BAD_SIZE;
-  if (act != 0 && act != 1) return LLMI_ERR_UNSUPPORTED;
+  if (act < 0 || act > 2) return LLMI_ERR_UNSUPPORTED;
+  const GateConstants gc{alpha, limit};
   const size_t total = (size_t)n_rows * inner;
   const int threads = 256;
   const size_t most = (size_t)sm_count() * 16;       // a grid-stride loop takes the rest
   const int blocks = (int)((total + threads - 1) / threads < most ? (total + threads - 1) / threads : most);
-  if (dtype == LLMI_DTYPE_F32)
-    return act == 0 ? launch_pdl(PDL_SMALL, swiglu_kernel<float, 0>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, inner, total)
-                    : launch_pdl(PDL_SMALL, swiglu_kernel<float, 1>, blocks, threads, 0, stream, (const float*)gate_up, (float*)out, inner, total);
-  else if (dtype == LLMI_DTYPE_BF16)
-    return act == 0 ? launch_pdl(PDL_SMALL, swiglu_kernel<__nv_bfloat16, 0>, blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up,
-                                 (__nv_bfloat16*)out, inner, total)
-                    : launch_pdl(PDL_SMALL, swiglu_kernel<__nv_bfloat16, 1>, blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up,
-                                 (__nv_bfloat16*)out, inner, total);
-  else
-    return LLMI_ERR_BAD_DTYPE;
-  return launch_status();
+  if (dtype == LLMI_DTYPE_F32) return launch_swiglu<float>(gate_up, out, inner, act, total, gc, blocks, threads, stream);
+  if (dtype == LLMI_DTYPE_BF16) return launch_swiglu<__nv_bfloat16>(gate_up, out, inner, act, total, gc, blocks, threads, stream);
+  return LLMI_ERR_BAD_DTYPE;
 }
 
 LLMI_EXPORT int llmi_activate(int dtype, const void* x, void* out, long total, int act, cudaStream_t stream) {

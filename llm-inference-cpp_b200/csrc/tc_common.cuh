@@ -68,6 +68,8 @@ struct TcParams {
   int* tickets;             // [tiles], zero before and after the launch
   int* error_flag;
   int act;                  // the gate's activation in mode OUT_SWIGLU (see gated_value); in mode OUT_STORE 2: relu(v)^2 is stored
+  const float* oscale;      // [m_out] or null: the value with its bias is multiplied by it (not in mode OUT_SWIGLU)
+  GateConstants gate;
 };
 
 // The epilogue of one thread: v holds 16 consecutive tokens (n_base..) of out feature m.  Called by all
@@ -79,6 +81,11 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, float* v, i
     // two halves of silu(gate) * up (src/model/transformer.cpp:290; src/model/kernels.cpp:148).  The even
     // lane finishes tokens 0..7 of the pair, the odd lane tokens 8..15.
     const bool is_gate = (m & 1) == 0;
+    if (p.bias) {                                            // a row's own bias, before the exchange
+      const float b = m < p.m_out ? p.bias[m] : 0.f;
+#pragma unroll
+      for (int c = 0; c < 16; ++c) v[c] += b;
+    }
     __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)n_base * p.ldo + (m >> 1);
 #pragma unroll
     for (int c = 0; c < 8; ++c) {
@@ -87,12 +94,12 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, float* v, i
       const float g = is_gate ? v[c] : recv, u = is_gate ? recv : v[c + 8];
       const int tok = is_gate ? c : c + 8;
       if (tok < n_valid && m < p.m_out)
-        o[(size_t)tok * p.ldo] = __float2bfloat16_rn(gated_value(g, u, p.act));
+        o[(size_t)tok * p.ldo] = __float2bfloat16_rn(gated_value(g, u, p.act, p.gate));
     }
     return;
   }
   if (m >= p.m_out) return;
-  const float b = p.bias ? p.bias[m] : 0.f;
+  const float b = p.bias ? p.bias[m] : 0.f, os = p.oscale ? p.oscale[m] : 1.f;
   if (p.mode == OUT_ADD_F32) {
     // One-way additions at the L2 (a reduction, nothing comes back): nobody else adds to these elements during the
     // launch, so the result is the one of read, add, store — without the read's round trip, which costs microseconds
@@ -100,13 +107,13 @@ __device__ __forceinline__ void tc_epilogue_store(const TcParams& p, float* v, i
     float* o = (float*)p.out + (size_t)n_base * p.ldo + m;
 #pragma unroll
     for (int c = 0; c < 16; ++c)
-      if (c < n_valid) asm volatile("red.global.add.f32 [%0], %1;" ::"l"(o + (size_t)c * p.ldo), "f"(v[c] + b) : "memory");
+      if (c < n_valid) asm volatile("red.global.add.f32 [%0], %1;" ::"l"(o + (size_t)c * p.ldo), "f"((v[c] + b) * os) : "memory");
     return;
   }
 #pragma unroll
   for (int c = 0; c < 16; ++c) {
     if (c >= n_valid) break;
-    const float val = v[c] + b;
+    const float val = (v[c] + b) * os;
     const size_t idx = (size_t)(n_base + c) * p.ldo + m;
     if (p.mode == OUT_STORE) ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16_rn(stored_value(val, p.act));
     else ((float*)p.out)[idx] = val;

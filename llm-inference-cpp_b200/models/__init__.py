@@ -1,2 +1,2 @@
 """Architectures this library knows; importing the package registers them."""
-from . import fusazen, garodra, gemosun, llama, renitar, zomurax  # noqa: F401
+from . import fusazen, garodra, gemosun, llama, renitar, sobezen, zomurax  # noqa: F401

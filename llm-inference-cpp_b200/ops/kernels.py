@@ -23,7 +23,8 @@ OUT_SWIGLU = 3       # y (compute type) = silu(gate)·up, W's rows alternating g
 OUT_GEGLU = 4        # the same with the tanh form of GELU as the gate's activation
 OUT_RELU2 = 5        # y (compute type) = relu(x·Wᵀ + bias)², the activation finished in the product's epilogue
 OUT_GELU = 6         # y (compute type) = gelu(x·Wᵀ + bias), the exact form v·Phi(v), finished in the product's epilogue
-_GATED = (OUT_SWIGLU, OUT_GEGLU)
+OUT_BOUNDED = 7      # as OUT_SWIGLU with the bounded gate: g from above at a limit, u on both sides, g · logistic(alpha g) · (u + 1)
+_GATED = (OUT_SWIGLU, OUT_GEGLU, OUT_BOUNDED)
 _STORES = (OUT_STORE, OUT_RELU2, OUT_GELU)      # the modes whose output has the compute type and the weight's row count
 
 _ERRORS = {
@@ -164,7 +165,8 @@ def lib():
                      "llmi_layernorm", "llmi_depth_mix", "llmi_gate_rows", "llmi_pool_rows", "llmi_mix_layernorm",
                      "llmi_moe_identity_add", "llmi_channel_decay", "llmi_rows_activate", "llmi_decay_recurrence",
                      "llmi_normed_pair", "llmi_stream_axpy_norm", "llmi_stream_postnorm", "llmi_softcap_rows", "llmi_moe_table",
-                     "llmi_qkv_unit_prepare", "llmi_latent_prepare_direct"):
+                     "llmi_qkv_unit_prepare", "llmi_latent_prepare_direct", "llmi_channel_token_supported",
+                     "llmi_channel_token_prepare", "llmi_channel_token_step", "llmi_cast_rows"):
             getattr(l, name).restype = c_int
         l.llmi_gemm_tc_workspace.restype = c_long
         l.llmi_delta_state_floats.restype = c_long
@@ -175,7 +177,7 @@ def lib():
         # The launchers of a prompt's step are called a few hundred times per step from Python: with their argument
         # types declared, plain integers go in without a ctypes object being made for each (a third of a call's cost).
         P, L, I, F = c_void_p, c_long, c_int, c_float
-        l.llmi_gemm_tc.argtypes = [P, L, P, L, P, P, L, I, I, I, I, P, L, P, I, P, P]
+        l.llmi_gemm_tc.argtypes = [P, L, P, L, P, P, L, I, I, I, I, P, L, P, I, P, P, F, F, P]
         l.llmi_rmsnorm.argtypes = [I, P, P, P, P, I, I, F, P]
         l.llmi_rope_store.argtypes = [I, P, L, P, I, P, P, P, I, I, P, P, I, I, I, I, I, P]
         l.llmi_attention_prefill_tc.argtypes = [P, L, L, P, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, I, P, L, P, I, P, I, P, P, L, P, I, P, L, P, P, P, P]
@@ -259,24 +261,33 @@ def gate_rows(a: torch.Tensor, z: torch.Tensor) -> None:
                                              c_long(z.stride(0)), c_int(T), _stream()))
 
 
-ACT_SILU, ACT_GELU_TANH = 0, 1
-ACTIVATIONS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH}
+ACT_SILU, ACT_GELU_TANH, ACT_BOUNDED = 0, 1, 2
+ACTIVATIONS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "bounded": ACT_BOUNDED}
 EXPERT_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "gelu": 3}      # of the routed experts' kernels (relu2: the square of relu; gelu: the exact form)
-FUSED_GATE_MODES = {ACT_SILU: OUT_SWIGLU, ACT_GELU_TANH: OUT_GEGLU}     # activation -> the output mode of the products that gate in their epilogue
+FUSED_GATE_MODES = {ACT_SILU: OUT_SWIGLU, ACT_GELU_TANH: OUT_GEGLU, ACT_BOUNDED: OUT_BOUNDED}     # activation -> the output mode of the products that gate in their epilogue
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU) -> None:
-    """out = act(gate_up[:, :F]) * gate_up[:, F:]; act: silu or the tanh form of GELU."""
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU, constants: tuple = (0.0, 0.0)) -> None:
+    """out = act(gate_up[:, :F]) * gate_up[:, F:]; act: silu or the tanh form of GELU.  ACT_BOUNDED with ``constants`` =
+    (alpha, limit): g = min(gate, limit), u = clamp(up, -limit, limit), out = g * logistic(alpha * g) * (u + 1)."""
     _need_cuda(gate_up, out)
     n, F = out.shape
     assert gate_up.shape == (n, 2 * F) and gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype
-    _check("swiglu", lib().llmi_swiglu(c_int(_dtype_code(out)), _ptr(gate_up), _ptr(out), c_int(n), c_int(F), c_int(act), _stream()))
+    _check("swiglu", lib().llmi_swiglu(c_int(_dtype_code(out)), _ptr(gate_up), _ptr(out), c_int(n), c_int(F), c_int(act),
+                                       c_float(constants[0]), c_float(constants[1]), _stream()))
+
+
+def _check_oscale(oscale, n: int, mode: int) -> None:
+    if oscale is not None:
+        assert mode not in _GATED and oscale.is_cuda and oscale.dtype == torch.float32 and oscale.numel() == n and oscale.is_contiguous()
 
 
 def linear_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None,
-                mode: int = OUT_STORE) -> None:
-    """out (mode) x·wᵀ + bias with fp32 FMA arithmetic; x [M,K], w [N,K], rows may be strided."""
+                mode: int = OUT_STORE, oscale: torch.Tensor | None = None) -> None:
+    """out (mode) (x·wᵀ + bias) * oscale with fp32 FMA arithmetic; x [M,K], w [N,K], rows may be strided; bias and oscale
+    fp32 [N], optional."""
     _need_cuda(x, w, out, bias)
+    _check_oscale(oscale, w.shape[0], mode)
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.shape == (M, N) and x.dtype == w.dtype
@@ -288,7 +299,7 @@ def linear_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.numel() == N
     _check("linear_simt", lib().llmi_linear_simt(
-        c_int(_dtype_code(x)), _ptr(x), c_long(x.stride(0)), _ptr(w), c_long(w.stride(0)), _ptr(bias), _ptr(out),
+        c_int(_dtype_code(x)), _ptr(x), c_long(x.stride(0)), _ptr(w), c_long(w.stride(0)), _ptr(bias), _ptr(oscale), _ptr(out),
         c_long(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(mode), _stream()))
 
 
@@ -343,9 +354,11 @@ def gemm_tc_eligible(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None,
-            mode: int = OUT_STORE) -> None:
-    """out (mode) x·wᵀ + bias on the tcgen05 tensor cores; bf16 inputs, fp32 accumulation."""
+            mode: int = OUT_STORE, oscale: torch.Tensor | None = None, constants: tuple = (0.0, 0.0)) -> None:
+    """out (mode) (x·wᵀ + bias) * oscale on the tcgen05 tensor cores; bf16 inputs, fp32 accumulation.  ``constants``: of the
+    gate in mode OUT_BOUNDED (see :func:`swiglu`); the bias of a gated mode alternates as w's rows do."""
     _need_cuda(x, w, out, bias)
+    _check_oscale(oscale, w.shape[0], mode)
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.shape == (M, N // 2 if mode in _GATED else N)
@@ -356,7 +369,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Ten
     sc = tc_scratch(x.device)
     _check("gemm_tc", lib().llmi_gemm_tc(
         x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), _addr(bias), out.data_ptr(), out.stride(0), M, N, K, mode,
-        sc.workspace.data_ptr(), sc.WORKSPACE_BYTES, sc.tickets.data_ptr(), sc.N_TICKETS, sc.error.data_ptr(), _stream_int()))
+        sc.workspace.data_ptr(), sc.WORKSPACE_BYTES, sc.tickets.data_ptr(), sc.N_TICKETS, sc.error.data_ptr(), _addr(oscale),
+        constants[0], constants[1], _stream_int()))
 
 
 class DeferredNorm:
@@ -387,7 +401,8 @@ class DeferredNorm:
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None,
-                mode: int = OUT_STORE, then_norm: DeferredNorm | None = None, scale_from: DeferredNorm | None = None) -> None:
+                mode: int = OUT_STORE, then_norm: DeferredNorm | None = None, scale_from: DeferredNorm | None = None,
+                oscale: torch.Tensor | None = None, constants: tuple = (0.0, 0.0)) -> None:
     """The same product for at most 64 tokens: the weight-streaming kernel (``csrc/gemm_skinny.cu``).
 
     ``then_norm`` (mode OUT_ADD_F32): also fill that deferred norm from the updated ``out``.
@@ -403,6 +418,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch
     if then_norm is not None:
         assert mode == OUT_ADD_F32 and then_norm.h.shape == (M, N) and then_norm.h.dtype == torch.bfloat16
         assert then_norm.weight.numel() == N and then_norm.h.stride(1) == 1
+    _check_oscale(oscale, N, mode)
     if scale_from is not None:
         assert scale_from.h.data_ptr() == x.data_ptr() and scale_from.h.shape == (M, K)
     sc = tc_scratch(x.device)
@@ -414,7 +430,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch
         c_int(M), c_int(N), c_int(K), c_int(mode),
         _ptr(e.weight if e else None), _ptr(e.h if e else None), c_long(e.h.stride(0) if e else 0), _ptr(e.ss if e else None),
         _ptr(f.ss if f else None), c_int(f.n_tiles if f else 0), c_float(f.eps if f else 0.0),
-        _ptr(sc.error), _stream()))
+        _ptr(sc.error), _ptr(oscale), c_float(constants[0]), c_float(constants[1]), _stream()))
 
 
 SKINNY_MAX_TOKENS = 16
@@ -449,13 +465,14 @@ def norm_deferrable(n_tokens: int, width: int, dtype) -> bool:
                 and n_tokens <= DeferredNorm.SS_STRIDE and width % 64 == 0)
 
 
-def gemm_bf16(x, w, out, bias=None, mode: int = OUT_STORE, then_norm: DeferredNorm | None = None) -> bool:
+def gemm_bf16(x, w, out, bias=None, mode: int = OUT_STORE, then_norm: DeferredNorm | None = None, oscale=None,
+              constants: tuple = (0.0, 0.0)) -> bool:
     """The bf16 tensor-core product: the weight-streaming kernel for a handful of tokens, the tcgen05
     kernel for more.  ``x`` may be a filled :class:`DeferredNorm`; returns whether ``then_norm`` was filled."""
     pending = x if isinstance(x, DeferredNorm) else None
     xin = pending.h if pending is not None else x
     if skinny_applies(xin, w):
-        gemm_skinny(xin, w, out, bias, mode, then_norm, pending)
+        gemm_skinny(xin, w, out, bias, mode, then_norm, pending, oscale, constants)
         return then_norm is not None
     if pending is not None:
         # this reader cannot apply the scale to its accumulators: the norm is run the plain way after all, over the
@@ -463,26 +480,27 @@ def gemm_bf16(x, w, out, bias=None, mode: int = OUT_STORE, then_norm: DeferredNo
         if pending.source is None:
             raise KernelError("a deferred norm that no product has filled")
         rmsnorm(pending.source, pending.weight, pending.h, pending.eps)
-    gemm_tc(xin, w, out, bias, mode)
+    gemm_tc(xin, w, out, bias, mode, oscale, constants)
     return False
 
 
-def linear(x, w, out, bias=None, mode: int = OUT_STORE, then_norm: DeferredNorm | None = None) -> bool:
+def linear(x, w, out, bias=None, mode: int = OUT_STORE, then_norm: DeferredNorm | None = None, oscale=None) -> bool:
     """The matrix product of the step: the tensor-core kernels for bf16 operands they can take (16-byte
     aligned rows), the fp32 FMA kernel for the 32-bit path and for everything else.  ``x`` may be a filled
-    :class:`DeferredNorm`; returns whether ``then_norm`` was filled (False: run that norm the plain way)."""
+    :class:`DeferredNorm`; returns whether ``then_norm`` was filled (False: run that norm the plain way).  ``oscale`` (fp32,
+    one number per row of w): the product with its bias is multiplied by it before it is stored or added."""
     xin = x.h if isinstance(x, DeferredNorm) else x
     if not _FORCE_SIMT and gemm_tc_eligible(xin, w):
-        return gemm_bf16(x, w, out, bias, mode, then_norm)
+        return gemm_bf16(x, w, out, bias, mode, then_norm, oscale)
     if isinstance(x, DeferredNorm):      # a reader that cannot scale: the norm the plain way after all
         if x.source is None:
             raise KernelError("a deferred norm that no product has filled")
         rmsnorm(x.source, x.weight, x.h, x.eps)
     if mode in _STORE_ACTIVATIONS:       # the fp32 FMA product has no activation in its epilogue: two steps
-        linear_simt(xin, w, out, bias, OUT_STORE)
+        linear_simt(xin, w, out, bias, OUT_STORE, oscale)
         activate(out, out, _STORE_ACTIVATIONS[mode])
         return False
-    linear_simt(xin, w, out, bias, mode)
+    linear_simt(xin, w, out, bias, mode, oscale)
     return False
 
 
@@ -1279,24 +1297,27 @@ def linear_batched(x: torch.Tensor, bx: int, w: torch.Tensor, out: torch.Tensor,
 # Latent attention
 
 def latent_prepare(down: torch.Tensor, Q: int, C: int, R: int, wq, wc, eps: float, inv_freq, rot_dims: int, ctx, seq_pages,
-                   page_size: int, cache: torch.Tensor, cq: torch.Tensor, write_kv: bool = True, pairing: int = 1) -> None:
+                   page_size: int, cache: torch.Tensor, cq: torch.Tensor, write_kv: bool = True, pairing: int = 1,
+                   amplitude: float = 1.0) -> None:
     """From the fp32 down-projection rows [query latent Q | latent C | shared key part R]: the RMS-normed query
     latent into ``cq`` (compute type) and the cache row [normed latent | rotated key part] of every token.  ``pairing``:
-    which entries turn together, 1 neighbours (2i, 2i + 1), 0 entries (i, i + rot_dims/2)."""
+    which entries turn together, 1 neighbours (2i, 2i + 1), 0 entries (i, i + rot_dims/2); cos and sin times ``amplitude``.
+    Without ``write_kv`` the rows may end behind the query latent (``wc`` None): nothing goes to the cache."""
     _need_cuda(down, wq, wc, inv_freq, seq_pages, cache, cq)
     T = down.shape[0]
-    assert down.dtype == torch.float32 and down.stride(1) == 1 and down.shape[1] >= Q + C + R
+    assert down.dtype == torch.float32 and down.stride(1) == 1 and down.shape[1] >= Q + (C + R if write_kv else 0)
     assert cq.shape == (T, Q) and cq.is_contiguous() and cq.dtype == cache.dtype and cache.is_contiguous()
-    assert cache.shape[-1] == C + R and cache.shape[-3] == 1 and wq.dtype == torch.float32 and wc.dtype == torch.float32
+    assert cache.shape[-1] == C + R and cache.shape[-3] == 1 and wq.dtype == torch.float32
+    assert not write_kv or wc.dtype == torch.float32
     _check("latent_prepare", lib().llmi_latent_prepare(
         c_int(_dtype_code(cq)), _ptr(down), c_long(down.stride(0)), c_int(Q), c_int(C), c_int(R), _ptr(wq), _ptr(wc), c_float(eps),
         _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(seq_pages), c_int(seq_pages.stride(0)),
-        c_int(page_size), _ptr(cache), _ptr(cq), c_int(T), c_int(1 if write_kv else 0), c_int(pairing), _stream()))
+        c_int(page_size), _ptr(cache), _ptr(cq), c_int(T), c_int(1 if write_kv else 0), c_int(pairing), c_float(amplitude), _stream()))
 
 
 def latent_prepare_direct(proj: torch.Tensor, H: int, D: int, C: int, R: int, wc, eps: float, inv_freq, rot_dims: int, pairing: int, ctx,
                           seq_pages, page_size: int, cache: torch.Tensor, qn: torch.Tensor, qa: torch.Tensor,
-                          write_kv: bool = True) -> None:
+                          write_kv: bool = True, amplitude: float = 1.0) -> None:
     """The same for queries that come straight from the layer's input: from the fp32 rows [q: H*(D+R) | latent C | shared
     key part R], the plain part of every head's query into ``qn`` [T, H*D], its rotated part behind the C leading entries
     of the head's row of ``qa`` [T, H*(C+R)], and the cache row of every token."""
@@ -1310,11 +1331,11 @@ def latent_prepare_direct(proj: torch.Tensor, H: int, D: int, C: int, R: int, wc
         c_int(_dtype_code(qn)), _ptr(proj), c_long(proj.stride(0)), c_int(H), c_int(D), c_int(C), c_int(R), _ptr(wc), c_float(eps),
         _ptr(inv_freq), c_int(rot_dims), c_int(pairing), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(seq_pages),
         c_int(seq_pages.stride(0)), c_int(page_size), _ptr(cache), _ptr(qn), _ptr(qa), c_long(qa.stride(0)), c_int(T),
-        c_int(1 if write_kv else 0), _stream()))
+        c_int(1 if write_kv else 0), c_float(amplitude), _stream()))
 
 
 def latent_q_rotate(q: torch.Tensor, D: int, qa: torch.Tensor, C: int, R: int, H: int, inv_freq, rot_dims: int, ctx,
-                    pairing: int = 1) -> None:
+                    pairing: int = 1, amplitude: float = 1.0) -> None:
     """The part of every head's query that is rotated by position, q[:, h, D:], into qa[:, h, C:]."""
     _need_cuda(q, qa, inv_freq)
     T = q.shape[0]
@@ -1322,7 +1343,7 @@ def latent_q_rotate(q: torch.Tensor, D: int, qa: torch.Tensor, C: int, R: int, H
     assert q.shape[1] == H * (D + R) and qa.shape == (T, H * (C + R))
     _check("latent_q_rotate", lib().llmi_latent_q_rotate(
         c_int(_dtype_code(q)), _ptr(q), c_long(q.stride(0)), c_int(D), _ptr(qa), c_long(qa.stride(0)), c_int(C), c_int(R), c_int(H),
-        _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), c_int(T), c_int(pairing), _stream()))
+        _ptr(inv_freq), c_int(rot_dims), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), c_int(T), c_int(pairing), c_float(amplitude), _stream()))
 
 
 _LATENT_ATTENTION = os.environ.get("LLMI_LATENT_ATTENTION", "mma")      # "generic": the fp32-arithmetic kernel for everything
@@ -1385,30 +1406,37 @@ def delta_state_floats(H: int, Hk: int, D: int, Dv: int, taps: int) -> int:
 
 
 def delta_step(proj: torch.Tensor, dims, conv_w, a_log, dt_bias, state: torch.Tensor, ctx, prep: torch.Tensor,
-               o_raw: torch.Tensor, write_state: bool = True) -> None:
+               o_raw: torch.Tensor, write_state: bool = True, z: torch.Tensor | None = None) -> None:
     """The recurrent part of a gated-delta-rule mixer for one step.  ``proj`` fp32 [T, .]: [q | k | v | b | a | gate]
     rows; ``dims = (H, Hk, D, Dv, taps)``; ``state`` [slots, state_floats] fp32 (read, and updated if
-    ``write_state``); ``prep`` fp32 [T, 2*Hk*D + H*Dv + 2*H] scratch; ``o_raw`` fp32 [T, H*Dv] receives S^T q."""
-    _need_cuda(proj, conv_w, a_log, dt_bias, state, prep, o_raw)
+    ``write_state``); ``prep`` fp32 [T, 2*Hk*D + H*Dv + 2*H] scratch; ``o_raw`` fp32 [T, H*Dv] receives S^T q.  With ``z``
+    fp32 [T, H*D] the decay is one per key channel, exp(-exp(a_log) * softplus(z + dt_bias)) with ``dt_bias`` [H*D]; the
+    rows are then [q | k | v | b | ...] and ``prep`` is [T, >= 2*Hk*D + H*Dv + H*D + H]."""
+    _need_cuda(proj, conv_w, a_log, dt_bias, state, prep, o_raw, z)
     H, Hk, D, Dv, taps = dims
     T = proj.shape[0]
     n_conv = 2 * Hk * D + H * Dv
     assert proj.dtype == prep.dtype == o_raw.dtype == state.dtype == torch.float32 and proj.stride(1) == 1
-    assert proj.shape[1] == n_conv + 2 * H + H * Dv and prep.shape == (T, n_conv + 2 * H) and o_raw.shape == (T, H * Dv)
-    assert prep.is_contiguous() and o_raw.is_contiguous() and state.is_contiguous() and conv_w.shape == (n_conv, taps)
-    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and a_log.numel() == H and dt_bias.numel() == H
+    if z is None:
+        assert proj.shape[1] == n_conv + 2 * H + H * Dv and prep.shape == (T, n_conv + 2 * H) and dt_bias.numel() == H
+    else:
+        assert proj.shape[1] >= n_conv + H and prep.shape[0] == T and prep.shape[1] >= n_conv + H * D + H and dt_bias.numel() == H * D
+        assert z.dtype == torch.float32 and z.shape == (T, H * D) and z.stride(1) == 1
+    assert o_raw.shape == (T, H * Dv) and prep.is_contiguous() and o_raw.is_contiguous() and state.is_contiguous()
+    assert conv_w.shape == (n_conv, taps) and conv_w.dtype == torch.float32 and conv_w.is_contiguous() and a_log.numel() == H
     assert state.shape[-1] == delta_state_floats(H, Hk, D, Dv, taps)
     l = lib()
     d = (c_int(H), c_int(Hk), c_int(D), c_int(Dv), c_int(taps))
     _check("delta_prepare", l.llmi_delta_prepare(_ptr(proj), c_long(proj.stride(0)), *d, _ptr(conv_w), _ptr(a_log), _ptr(dt_bias),
                                                  _ptr(state), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_q_start),
-                                                 _ptr(ctx.seq_slot), _ptr(prep), c_long(prep.stride(0)), c_int(T), _stream()))
+                                                 _ptr(ctx.seq_slot), _ptr(prep), c_long(prep.stride(0)), c_int(T), _ptr(z),
+                                                 c_long(z.stride(0) if z is not None else 0), _stream()))
     if write_state and taps > 1:
         _check("delta_conv_carry", l.llmi_delta_conv_carry(_ptr(proj), c_long(proj.stride(0)), *d, _ptr(state), _ptr(ctx.seq_q_start),
                                                            _ptr(ctx.seq_kv_len), _ptr(ctx.seq_slot), c_int(ctx.n_seqs), _stream()))
     _check("delta_recurrence", l.llmi_delta_recurrence(_ptr(prep), c_long(prep.stride(0)), *d, _ptr(state), _ptr(ctx.seq_q_start),
                                                        _ptr(ctx.seq_slot), _ptr(o_raw), c_long(o_raw.stride(0)), c_int(ctx.n_seqs),
-                                                       c_int(1 if write_state else 0), _stream()))
+                                                       c_int(1 if write_state else 0), c_int(1 if z is not None else 0), _stream()))
 
 
 GATE_SILU, GATE_SIGMOID = 0, 1
@@ -1428,6 +1456,57 @@ def delta_finish(o_raw: torch.Tensor, gate: torch.Tensor, weight, eps: float, H:
                                                    c_long(gate.stride(0)), _ptr(weight), c_int(per_head), c_int(gate_act),
                                                    c_float(eps), c_int(H), c_int(Dv), _ptr(ctx.tok_seq), _ptr(out),
                                                    c_long(out.stride(0)), c_int(T), _stream()))
+
+
+# ---------------------------------------------------------------------------------------------
+# The gated delta rule with a decay per key channel: steps of single tokens (csrc/channel_delta.cu)
+
+def channel_token_supported(dims, rank_a: int, rank_g: int) -> bool:
+    return bool(lib().llmi_channel_token_supported(*(c_int(d) for d in dims), c_int(rank_a), c_int(rank_g)))
+
+
+def channel_token(proj: torch.Tensor, dims, low_a: tuple, low_g: tuple, conv_w, a_log, dt_bias, w_a: torch.Tensor, w_g: torch.Tensor,
+                  state: torch.Tensor, ctx, prep: torch.Tensor, gate: torch.Tensor, weight, eps: float, out: torch.Tensor,
+                  write_state: bool = True) -> None:
+    """For a step in which every sequence brings one token, everything between the two products of a gated-delta-rule mixer
+    with a decay per key channel and a logistic output gate through low-rank paths (sizes: :func:`channel_token_supported`).
+    ``proj`` fp32 rows [q | k | v | b | ...] with the two low-rank vectors at ``low_a`` and ``low_g`` = (first column, size);
+    ``w_a`` [rank_a, H*D up to a multiple of 64], ``w_g`` [rank_g, H*Dv likewise]: the paths' second matrices, transposed,
+    zeros behind, in out's type.  ``prep`` fp32 [T, >= 2*Hk*D + H*Dv + H*D + H] (row pitch a multiple of four) and ``gate`` fp32
+    [T, H*Dv] are scratch; ``out`` [T, H*Dv] = o / rms(o) * weight * logistic(gate)."""
+    _need_cuda(proj, conv_w, a_log, dt_bias, w_a, w_g, state, prep, gate, weight, out)
+    H, Hk, D, Dv, taps = dims
+    T = proj.shape[0]
+    n_conv = 2 * Hk * D + H * Dv
+    assert proj.dtype == prep.dtype == gate.dtype == state.dtype == weight.dtype == torch.float32 and proj.stride(1) == 1
+    assert proj.shape[1] >= max(n_conv + H, low_a[0] + low_a[1], low_g[0] + low_g[1])
+    assert prep.stride(1) == 1 and prep.shape[1] >= n_conv + H * D + H and gate.shape == (T, H * Dv) and gate.stride(1) == 1
+    assert w_a.dtype == w_g.dtype == out.dtype and w_a.shape == (low_a[1], _up64(H * D)) and w_g.shape == (low_g[1], _up64(H * Dv))
+    assert w_a.is_contiguous() and w_g.is_contiguous() and conv_w.shape == (n_conv, taps) and conv_w.is_contiguous()
+    assert a_log.numel() == H and dt_bias.numel() == H * D and weight.numel() == Dv and out.shape == (T, H * Dv) and out.stride(1) == 1
+    assert state.is_contiguous() and state.shape[-1] == delta_state_floats(H, Hk, D, Dv, taps)
+    d = (c_int(H), c_int(Hk), c_int(D), c_int(Dv), c_int(taps))
+    l, code, wr = lib(), c_int(_dtype_code(out)), c_int(1 if write_state else 0)
+    _check("channel_token_prepare", l.llmi_channel_token_prepare(
+        code, _ptr(proj), c_long(proj.stride(0)), *d, c_int(low_a[0]), c_int(low_a[1]), c_int(low_g[0]), c_int(low_g[1]), _ptr(conv_w),
+        _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(ctx.tok_seq), _ptr(ctx.seq_slot), _ptr(w_a), _ptr(w_g), _ptr(prep),
+        c_long(prep.stride(0)), _ptr(gate), c_long(gate.stride(0)), c_int(T), wr, _stream()))
+    _check("channel_token_step", l.llmi_channel_token_step(
+        code, _ptr(prep), c_long(prep.stride(0)), *d, _ptr(state), _ptr(ctx.tok_seq), _ptr(ctx.seq_slot), _ptr(gate),
+        c_long(gate.stride(0)), _ptr(weight), c_float(eps), _ptr(out), c_long(out.stride(0)), c_int(T), wr, _stream()))
+
+
+def _up64(n: int) -> int:
+    return -(-n // 64) * 64
+
+
+def cast_rows(src: torch.Tensor, out: torch.Tensor) -> None:
+    """out [T, n] (contiguous, any compute type) = src, an fp32 view [T, n] with strided rows."""
+    _need_cuda(src, out)
+    T, n = out.shape
+    assert src.dtype == torch.float32 and src.shape == (T, n) and src.stride(1) == 1 and out.is_contiguous()
+    _check("cast_rows", lib().llmi_cast_rows(c_int(_dtype_code(out)), _ptr(src), c_long(src.stride(0)), _ptr(out), c_int(T), c_int(n),
+                                             _stream()))
 
 
 # ---------------------------------------------------------------------------------------------

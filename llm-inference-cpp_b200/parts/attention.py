@@ -351,7 +351,10 @@ class WindowPoolAttention(_MapsAttention):
 class GatedAttention(_MapsAttention):
     """Softmax attention of grouped queries with optional pieces, each a parameter:
 
-    * ``bias``: the q, k, v and output projections have biases (the tensor's name + ``.b``);
+    * ``bias``: the q, k, v and output projections have biases (the tensor's name + ``.b``); ``out_bias`` (default: as
+      ``bias``): whether the output projection has one;
+    * ``values_from_keys``: there is no value projection; the values are the keys as projected (with their bias), before
+      the rotation;
     * ``conv`` (taps; 0: none): a short causal convolution over time on every channel of q, k and v, right behind the
       projection: y[t] = sum_j w[:, j] * u[t - taps + 1 + j], zeros before the sequence's start, no bias, the input itself
       not added.  The last taps - 1 projected rows of a sequence are kept in the cache's state slab (fp32);
@@ -364,23 +367,28 @@ class GatedAttention(_MapsAttention):
     * ``gate``: every output entry is multiplied by logistic(W_g h) of its own, before the output projection.
 
     params: ``width``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale``, ``eps`` (of the q and k norms), and the
-    above.  tensors: ``q`` [heads*dim, width], ``k`` [kv_heads*dim, width], ``v`` [kv_heads*vdim, width], ``o`` [width,
-    heads*vdim]; with ``bias`` ``q.b``, ``k.b``, ``v.b``, ``o.b``; with ``conv`` ``q.conv``, ``k.conv``, ``v.conv``
+    above.  tensors: ``q`` [heads*dim, width], ``k`` [kv_heads*dim, width], ``v`` [kv_heads*vdim, width] (absent with
+    ``values_from_keys``), ``o`` [width, heads*vdim]; with ``bias`` ``q.b``, ``k.b``, ``v.b``, ``o.b``; with ``conv`` ``q.conv``, ``k.conv``, ``v.conv``
     [channels, taps]; with ``qk_norm`` ``q.norm``, ``k.norm``; with ``gate`` ``g`` [heads*vdim, width]."""
     stores_output = True
-    defers_norm = False
+    scales_output = True
 
     @classmethod
     def declare(cls, spec):
         p = spec.params
         d = cls._declare_projections(p, 1)
         H, G, D, Dv, W = p["heads"], p["kv_heads"], p["dim"], p["vdim"], p["width"]
+        sizes = {"q": H * D, "k": G * D}
+        if p.get("values_from_keys", False):
+            del d["v"]
+        else:
+            sizes["v"] = G * Dv
         if p.get("bias", False):
-            d.update({"q.b": TensorDecl((H * D,), "bias"), "k.b": TensorDecl((G * D,), "bias"),
-                      "v.b": TensorDecl((G * Dv,), "bias"), "o.b": TensorDecl((W,), "bias")})
+            d.update({n + ".b": TensorDecl((rows,), "bias") for n, rows in sizes.items()})
+        if p.get("out_bias", p.get("bias", False)):
+            d["o.b"] = TensorDecl((W,), "bias")
         if p.get("conv", 0):
-            K = p["conv"]
-            d.update({"q.conv": TensorDecl((H * D, K)), "k.conv": TensorDecl((G * D, K)), "v.conv": TensorDecl((G * Dv, K))})
+            d.update({n + ".conv": TensorDecl((rows, p["conv"])) for n, rows in sizes.items()})
         if p.get("qk_norm", False):
             d.update({"q.norm": TensorDecl((H * D,), "norm_scale"), "k.norm": TensorDecl((G * D,), "norm_scale")})
         if p.get("gate", False):
@@ -397,22 +405,28 @@ class GatedAttention(_MapsAttention):
         if self.shares_kv:
             raise ValueError("gated_attention: has key and value projections of its own")
         H, G, D, Dv = self.H, self.G, self.D, self.Dv
-        self.n_qkv = H * D + G * D + G * Dv
+        self.values_from_keys = bool(p.get("values_from_keys", False))
+        if self.values_from_keys and (Dv != D or p.get("conv", 0) or p.get("qk_norm", False)):
+            raise ValueError("gated_attention: values that are the keys have the keys' size and neither a convolution nor a norm")
+        qkv = ["q", "k"] + ([] if self.values_from_keys else ["v"])
+        self.n_qkv = H * D + G * D + (0 if self.values_from_keys else G * Dv)
         self.softcap = float(p.get("softcap", 0.0) or 0.0)
         self.gated = bool(p.get("gate", False))
         self.taps = int(p.get("conv", 0) or 0)
-        names = ["q", "k", "v"] + (["g"] if self.gated else [])
-        self.w_in = rt.to_compute(torch.cat([tensors[n] for n in names], dim=0))       # one product: [q | k | v | (gate)]
+        names = qkv + (["g"] if self.gated else [])
+        self.w_in = rt.to_compute(torch.cat([tensors[n] for n in names], dim=0))       # one product: [q | k | (v) | (gate)]
         self.w_o = rt.to_compute(tensors["o"])
         self.b_in = self.b_o = None
         if p.get("bias", False):
-            parts = [tensors["q.b"].float(), tensors["k.b"].float(), tensors["v.b"].float()]
+            parts = [tensors[n + ".b"].float() for n in qkv]
             if self.gated:
                 parts.append(torch.zeros(H * Dv, dtype=torch.float32, device=parts[0].device))
-            self.b_in, self.b_o = rt.to_f32(torch.cat(parts)), rt.to_f32(tensors["o.b"])
+            self.b_in = rt.to_f32(torch.cat(parts))
+        if p.get("out_bias", p.get("bias", False)):
+            self.b_o = rt.to_f32(tensors["o.b"])
         self.conv_w = None
         if self.taps:        # [taps, channels]: neighbouring channels side by side, the oldest tap first
-            self.conv_w = rt.to_f32(torch.cat([tensors[n + ".conv"] for n in ("q", "k", "v")], dim=0)).t().contiguous()
+            self.conv_w = rt.to_f32(torch.cat([tensors[n + ".conv"] for n in qkv], dim=0)).t().contiguous()
         if p.get("qk_norm", False):
             self.q_norm_w, self.k_norm_w = rt.to_f32(tensors["q.norm"]), rt.to_f32(tensors["k.norm"])
         self.pairing, self.amplitude = 0, 1.0
@@ -431,7 +445,7 @@ class GatedAttention(_MapsAttention):
     def weight_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o))
 
-    def forward(self, h, x, ctx, binding, store: bool = False, then_norm=None) -> bool:
+    def forward(self, h, x, ctx, binding, store: bool = False, then_norm=None, out_scale=None) -> bool:
         T = h.shape[0]
         rt, H, G, D, Dv = self.rt, self.H, self.G, self.D, self.Dv
         proj = rt.scratch("attn_proj", (T, self.w_in.shape[0]), torch.float32)
@@ -454,13 +468,13 @@ class GatedAttention(_MapsAttention):
         q = rt.scratch("attn_q", (T, H * D))
         kernels.qkv_prepare(qkv, H, G, D, G, Dv, self.q_norm_w, self.k_norm_w, self.eps, self.inv_freq, self.rot_dims, ctx, pages,
                             g.page_size, k_cache, v_cache, q, has_kv=True, write_kv=binding.writes, pairing=self.pairing,
-                            amplitude=self.amplitude)
+                            amplitude=self.amplitude, v_from_k=self.values_from_keys)
         out = rt.scratch("attn_out", (T, H * Dv))
         kernels.attention_maps(q, out, k_cache, v_cache, ctx, pages, g.page_size, H, G, 1, D, Dv, self.scale, None,
                                self.window, self.chunk, rt=rt, gate=proj[:, self.n_qkv:] if self.gated else None,
                                softcap=self.softcap)
-        kernels.linear(out, self.w_o, x, self.b_o, kernels.OUT_STORE_F32 if store else kernels.OUT_ADD_F32)
-        return False
+        return kernels.linear(out, self.w_o, x, self.b_o, kernels.OUT_STORE_F32 if store else kernels.OUT_ADD_F32,
+                              None if store else then_norm, out_scale)
 
 
 @part("mixer", "distance_attention")

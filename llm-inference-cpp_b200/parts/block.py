@@ -1,6 +1,7 @@
 """Arrangements of a layer.  ``prenorm``: x += mixer(norm(x)); x += ffn(norm(x))
 (include/llmi/model/transformer.hpp:49-52); the feed-forward may be absent, and a part in the slot ``mixer_conv``
-(family ``conv``) acts on the mixer's input: x += mixer(conv(norm(x))).
+(family ``conv``) acts on the mixer's input: x += mixer(conv(norm(x))).  Parts in the slots ``mixer_scale`` and ``ffn_scale``
+(family ``scale``) multiply what the two sublayers add, entry by entry.
 
 Norm deferral (optional, see :class:`ops.kernels.DeferredNorm`): a mixer or feed-forward whose class sets
 ``defers_norm = True`` accepts a filled deferred norm as its input ``h`` and a keyword ``then_norm`` — a
@@ -23,13 +24,19 @@ def _defers(p) -> bool:
 @part("block", "prenorm")
 class PreNormBlock:
     takes_padding_rows = True       # token rows of no sequence (a step padded to a shape) do no harm: rows are treated alone
-    def __init__(self, mixer_norm, mixer, ffn_norm=None, ffn=None, mixer_conv=None):
+    def __init__(self, mixer_norm, mixer, ffn_norm=None, ffn=None, mixer_conv=None, mixer_scale=None, ffn_scale=None):
         """``ffn_norm`` and ``ffn`` come together or not at all (a layer without a feed-forward); ``mixer_conv`` (a part
-        of the family ``conv``) reshapes what the mixer reads: x += mixer(conv(norm(x)))."""
+        of the family ``conv``) reshapes what the mixer reads: x += mixer(conv(norm(x))); ``mixer_scale`` and ``ffn_scale``
+        (parts of the family ``scale``): a factor per entry on what the sublayer adds (it must take ``out_scale=``)."""
         if (ffn is None) != (ffn_norm is None):
             raise ValueError("prenorm: a feed-forward comes with its norm, or not at all")
         self.mixer_norm, self.mixer, self.ffn_norm, self.ffn = mixer_norm, mixer, ffn_norm, ffn
         self.mixer_conv = mixer_conv
+        for p, s in ((mixer, mixer_scale), (ffn, ffn_scale)):
+            if s is not None and not getattr(p, "scales_output", False):
+                raise ValueError(f"prenorm: the part {getattr(p, 'kind', p)!r} cannot scale what it adds (out_scale=)")
+        self.mixer_extra = {} if mixer_scale is None else {"out_scale": mixer_scale.weight}
+        self.ffn_extra = {} if ffn_scale is None else {"out_scale": ffn_scale.weight}
 
     @property
     def entry_norm(self):
@@ -52,22 +59,30 @@ class PreNormBlock:
         else:
             h = entry if isinstance(entry, kernels.DeferredNorm) else self.mixer_norm.forward(x)
         if self.ffn is None:
-            self.mixer.forward(h, x, ctx, binding)
-            return None
+            return self._alone(h, x, ctx, binding, next_norm)
         then = None
         if _defers(self.mixer) and _defers(self.ffn) and hasattr(self.ffn_norm, "deferred"):
             then = self.ffn_norm.deferred(T, "deferred_inner")
-        if then is not None and self.mixer.forward(h, x, ctx, binding, then_norm=then):
+        if then is not None and self.mixer.forward(h, x, ctx, binding, then_norm=then, **self.mixer_extra):
             h = then
         else:
             if then is None:
-                self.mixer.forward(h, x, ctx, binding)
+                self.mixer.forward(h, x, ctx, binding, **self.mixer_extra)
             h = self.ffn_norm.forward(x)
         then = next_norm.deferred(T, "deferred_outer") if (hasattr(next_norm, "deferred") and _defers(self.ffn)) else None
         if then is not None:
-            return then if self.ffn.forward(h, x, ctx, then_norm=then) else None
-        self.ffn.forward(h, x, ctx)
+            return then if self.ffn.forward(h, x, ctx, then_norm=then, **self.ffn_extra) else None
+        self.ffn.forward(h, x, ctx, **self.ffn_extra)
         return None
+
+    def _alone(self, h, x, ctx, binding, next_norm):
+        """A layer without a feed-forward: the mixer's product is the one that may fill the next block's norm."""
+        then = (next_norm.deferred(x.shape[0], "deferred_outer")
+                if (hasattr(next_norm, "deferred") and _defers(self.mixer)) else None)
+        if then is None:
+            self.mixer.forward(h, x, ctx, binding, **self.mixer_extra)
+            return None
+        return then if self.mixer.forward(h, x, ctx, binding, then_norm=then, **self.mixer_extra) else None
 
 
 @part("block", "parallel")

@@ -7,7 +7,7 @@ the parts appear.
 """
 from __future__ import annotations
 
-from . import attention, block, conv, decay, delta, depth, embedding, experts, feedforward, latent, loop, norm, position, sidebyside  # noqa: F401  (register the built-in parts)
+from . import attention, block, conv, decay, delta, depth, embedding, experts, feedforward, latent, loop, norm, position, scale, sidebyside  # noqa: F401  (register the built-in parts)
 from .registry import TensorDecl, get_part
 from .spec import ModelSpec, PartSpec
 

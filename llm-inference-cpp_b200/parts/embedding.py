@@ -52,7 +52,8 @@ class TokenTable:
 @part("head", "linear_head")
 class LinearHead:
     """params: ``vocab``, ``width``, ``tied``, optional ``tensor`` (the matrix's local name; default ``weight``),
-    optional ``softcap`` (0: none; a logit z becomes softcap * tanh(z / softcap)).  tensors: the matrix [vocab, width] unless tied."""
+    optional ``softcap`` (0: none; a logit z becomes softcap * tanh(z / softcap)), optional ``scale`` (the logits are
+    multiplied by it, before the cap; default 1).  tensors: the matrix [vocab, width] unless tied."""
     takes_padding_rows = True       # token rows of no sequence (a step padded to a shape) do no harm: rows are treated alone
 
     @classmethod
@@ -65,6 +66,8 @@ class LinearHead:
         self.rt = rt
         self.vocab, self.width = int(spec.params["vocab"]), int(spec.params["width"])
         self.softcap = float(spec.params.get("softcap", 0.0) or 0.0)
+        scale = float(spec.params.get("scale", 1.0))
+        self.out_scale = torch.full((self.vocab,), scale, dtype=torch.float32, device=rt.device) if scale != 1.0 else None
         self.tied = bool(spec.params.get("tied", False))
         if self.tied:
             if embedding is None:
@@ -78,7 +81,7 @@ class LinearHead:
 
     def forward(self, h_rows):
         logits = self.rt.scratch("logits", (h_rows.shape[0], self.vocab), torch.float32)
-        kernels.linear(h_rows, self.weight, logits, None, kernels.OUT_STORE_F32)
+        kernels.linear(h_rows, self.weight, logits, None, kernels.OUT_STORE_F32, oscale=self.out_scale)
         if self.softcap > 0.0:
             kernels.softcap_rows(logits, self.softcap)
         return logits

@@ -32,6 +32,9 @@ Families and what the engine calls on their members (``rt`` is the
                its own place in the cache (``CacheBinding.more[slot]`` of the call).  Any part of a layer other than the
                mixer that has ``cache_request`` gets such a place
 
+``scale``      ``weight``: fp32 ``[width]``, a factor per entry on what a sublayer adds; the block hands it to a mixer or
+               feed-forward that sets ``scales_output`` as ``forward(..., out_scale=weight)``
+
 Every member also has ``declare(spec) -> {local tensor name: TensorDecl}`` (a
 classmethod: what it reads from the weight file under ``spec.prefix``) and is
 constructed as ``cls(spec, tensors, rt, **context)`` with its declared tensors.
@@ -60,7 +63,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass
 
-FAMILIES = ("norm", "position", "mixer", "ffn", "block", "embedding", "head", "pass_entry", "conv", "pass_exit")
+FAMILIES = ("norm", "position", "mixer", "ffn", "block", "embedding", "head", "pass_entry", "conv", "pass_exit", "scale")
 _PARTS: dict[str, dict[str, type]] = {f: {} for f in FAMILIES}
 
 
