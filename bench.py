@@ -2,11 +2,11 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
     python bench.py --workload smollm2-360m|smollm2-135m [--workload-dtypes bfloat16,float32]
-    python bench.py --design garodra|fusazen|gemosun|renitar|zomurax [--design-sizes 2048,1024]  (its own JSON line: that design's prefill and
-                                                                                  decode beside the Llama decoder (renitar: beside the
-                                                                                  Fusazen design, zomurax: beside the Garodra design) at
-                                                                                  equal size; garodra also has the size 2048-looped,
-                                                                                  zomurax the size 2048-full)
+    python bench.py --design garodra|fusazen|gemosun|renitar|zomurax|sobezen [--design-sizes 2048,1024]  (its own JSON line: that design's
+                                                                                  prefill and decode beside the Llama decoder (renitar:
+                                                                                  beside the Fusazen design, zomurax and sobezen: beside
+                                                                                  the Garodra design) at equal size; garodra also has the
+                                                                                  size 2048-looped, zomurax the size 2048-full)
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and context 4096 (a
 "step" is one decode step of the whole batch), timed on the device with CUDA events around
@@ -366,6 +366,41 @@ ZOMURAX_SIZES = {
 }
 
 
+# --design sobezen: the Sobezen design at sizes that resemble a real model's layers, beside the Garodra design (the closest
+# of the library's models: attention through a latent and a gated delta rule) at equal width, depth and feed-forward size.
+# Eight layers: latent attention with rows of its own, the delta rule with a decay per key channel (no feed-forward), attention
+# of grouped queries whose values are the keys, latent attention on the first layer's rows, and the same four again.  The
+# Garodra design beside it alternates its two mixers, with the dense feed-forward in every layer but every fourth.
+def sobezen_config(width, heads, kv_heads, dim, rot_dim, kv_rank, q_rank, ff, vocab, conv=4):
+    rot = {"base": 10000.0, "dims": rot_dim, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": kv_rank, "q_rank": q_rank,
+           "scale": (dim + rot_dim) ** -0.5, "rot": rot}
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": conv}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 10000.0, "dims": dim}}
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    layers = []
+    for first in (0, 4):
+        layers += [("latent_attention", lat, mlp), ("channel_delta", delta, None), ("attention", att, mlp),
+                   ("latent_attention", dict(lat, kv_from=first), mlp)]
+    return {"architecture": "Sobezen", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in layers]}
+
+
+def garodra_dense_config(width, heads, dim, rot_dim, kv_rank, q_rank, ff, vocab, conv=4):
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": kv_rank, "q_rank": q_rank,
+           "scale": (dim + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": conv}
+    kinds = [("latent_attention", lat), ("delta", delta)]
+    return {"architecture": "Garodra", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [{"type": kinds[i % 2][0], "mixer": kinds[i % 2][1], "mlp": None if i % 4 == 1 else {"kind": "dense", "ff": ff}} for i in range(8)]}
+
+
+SOBEZEN_SIZES = {
+    "2048": (sobezen_config(2048, 16, 4, 128, 64, 512, 1536, 8192, 49152), garodra_dense_config(2048, 16, 128, 64, 512, 1536, 8192, 49152), "garodra"),
+    "1024": (sobezen_config(1024, 8, 2, 64, 32, 256, 768, 4096, 49152), garodra_dense_config(1024, 8, 64, 32, 256, 768, 4096, 49152), "garodra"),
+}
+
+
 class KernelTimes:
     """Device time per entry point of ops.kernels inside real steps (CUDA events around every call; steps run launch
     by launch while this is on, so the figures are shares of a step, not a benchmark of it)."""
@@ -374,7 +409,7 @@ class KernelTimes:
              "moe_experts_streamed", "moe_experts_grouped", "conv_add", "qkv_prepare", "attention_maps", "diff_combine",
              "gdelta_prepare", "dplr_recurrence", "activate", "layernorm", "depth_mix", "pool_rows", "gate_rows", "tanh_rows",
              "channel_decay", "rows_silu", "decay_recurrence", "normed_pair", "stream_axpy_norm", "moe_identity_add",
-             "qkv_unit_prepare", "latent_prepare_direct", "moe_table", "stream_postnorm", "softcap_rows")
+             "qkv_unit_prepare", "latent_prepare_direct", "moe_table", "stream_postnorm", "softcap_rows", "channel_token", "cast_rows")
 
     def __init__(self):
         self.spans, self.saved = [], {}
@@ -418,7 +453,7 @@ def design_run(name, steps, warmup, batch, context, tokens, sizes):
     import llmi_b200 as L
     from llmi_b200 import SequenceStep
     tables = {"garodra": DESIGN_SIZES, "fusazen": FUSAZEN_SIZES, "gemosun": GEMOSUN_SIZES, "renitar": RENITAR_SIZES,
-              "zomurax": ZOMURAX_SIZES}
+              "zomurax": ZOMURAX_SIZES, "sobezen": SOBEZEN_SIZES}
     if name not in tables:
         print(f"bench.py: unknown design {name!r}")
         return 2
@@ -489,8 +524,9 @@ def main():
     ap.add_argument("--kv-heads", type=int, default=None,
                     help="with --only: another number of key/value heads (grouped queries), to profile their kernels")
     ap.add_argument("--design", default=None,
-                    help="'garodra', 'fusazen', 'gemosun', 'renitar' or 'zomurax': that design's prefill and decode throughput at layer sizes of a real model, beside the "
-                         "Llama decoder (renitar: beside the Fusazen design, zomurax: beside the Garodra design) at equal size (its own JSON line; the default workload is untouched)")
+                    help="'garodra', 'fusazen', 'gemosun', 'renitar', 'zomurax' or 'sobezen': that design's prefill and decode throughput at layer sizes of a real model, "
+                         "beside the Llama decoder (renitar: beside the Fusazen design, zomurax and sobezen: beside the Garodra design) at equal size (its own JSON line; the "
+                         "default workload is untouched)")
     ap.add_argument("--design-sizes", default="2048,1024", help="with --design: which of " + ", ".join(sorted(set(DESIGN_SIZES) | set(GEMOSUN_SIZES) | set(ZOMURAX_SIZES))))
     args = ap.parse_args()
 

@@ -137,7 +137,7 @@ delta_conv_carry_kernel(const float* __restrict__ proj, long ld, DeltaDims m, fl
   for (int j = 0; j < K - 1; ++j) carry[(size_t)j * Nc + ch] = keep[j];
 }
 
-// One block per (head, sequence), one thread per column j of S.  DREG > 0: the column (D = DREG entries) lives in
+// One block per (head, sequence, slice of columns), one thread per column j of S.  DREG > 0: the column (D = DREG entries) lives in
 // registers; DREG == 0: any D, the column lives in shared memory (S_s[d][j]: no two threads share a bank).
 // k and q of the next token are fetched while the current one is computed (two buffers, one barrier per token).
 template <int DREG>
@@ -154,8 +154,8 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
   const int r0 = seq_q_start[seq], n = seq_q_start[seq + 1] - r0;
   if (n <= 0) return;
   const int D = DREG > 0 ? DREG : m.D, Dv = m.Dv;
-  const int cols = blockDim.x;                               // Dv rounded up to whole warps
-  const int j = threadIdx.x;
+  const int cols = blockDim.x;                               // columns of a slice: whole warps
+  const int col = threadIdx.x, j = blockIdx.z * cols + col;
   const bool live = j < Dv;
   const int per = (m.channel ? 3 : 2) * D;
   float* kq = sm;                                            // [2][2*D]: k then q of a token (then its decays, if per channel)
@@ -168,7 +168,7 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
 #pragma unroll
       for (int d = 0; d < DREG; ++d) S_r[d] = S_g[(size_t)j * D + d];
     } else {
-      for (int d = 0; d < D; ++d) S_s[(size_t)d * cols + j] = S_g[(size_t)j * D + d];
+      for (int d = 0; d < D; ++d) S_s[(size_t)d * cols + col] = S_g[(size_t)j * D + d];
     }
   }
   auto fetch = [&](int i, int buf) {
@@ -191,15 +191,15 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
     if (m.channel) {
       const float* gd = q + D;
       for (int d = 0; d < D; ++d) {
-        const float s = gd[d] * S_s[(size_t)d * cols + j];
-        S_s[(size_t)d * cols + j] = s;
+        const float s = gd[d] * S_s[(size_t)d * cols + col];
+        S_s[(size_t)d * cols + col] = s;
         sk = fmaf(s, k[d], sk);
       }
       const float u = beta * (v - sk);
       float o = 0.f;
       for (int d = 0; d < D; ++d) {
-        const float s = fmaf(k[d], u, S_s[(size_t)d * cols + j]);
-        S_s[(size_t)d * cols + j] = s;
+        const float s = fmaf(k[d], u, S_s[(size_t)d * cols + col]);
+        S_s[(size_t)d * cols + col] = s;
         o = fmaf(s, q[d], o);
       }
       o_raw[(size_t)(r0 + i) * ldo + (size_t)h * Dv + j] = o;
@@ -210,7 +210,7 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
 #pragma unroll
       for (int d = 0; d < DREG; ++d) sk = fmaf(S_r[d], k[d], sk);
     } else {
-      for (int d = 0; d < D; ++d) sk = fmaf(S_s[(size_t)d * cols + j], k[d], sk);
+      for (int d = 0; d < D; ++d) sk = fmaf(S_s[(size_t)d * cols + col], k[d], sk);
     }
     const float u = beta * (v - g * sk);                     // (g S)ᵀ k = g (Sᵀ k)
     float o = 0.f;
@@ -223,8 +223,8 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
       }
     } else {
       for (int d = 0; d < D; ++d) {
-        const float s = fmaf(k[d], u, g * S_s[(size_t)d * cols + j]);
-        S_s[(size_t)d * cols + j] = s;
+        const float s = fmaf(k[d], u, g * S_s[(size_t)d * cols + col]);
+        S_s[(size_t)d * cols + col] = s;
         o = fmaf(s, q[d], o);
       }
     }
@@ -235,7 +235,7 @@ delta_recurrence_kernel(const float* __restrict__ prep, long ldp, DeltaDims m, f
 #pragma unroll
       for (int d = 0; d < DREG; ++d) S_g[(size_t)j * D + d] = S_r[d];
     } else {
-      for (int d = 0; d < D; ++d) S_g[(size_t)j * D + d] = S_s[(size_t)d * cols + j];
+      for (int d = 0; d < D; ++d) S_g[(size_t)j * D + d] = S_s[(size_t)d * cols + col];
     }
   }
 }
@@ -466,15 +466,18 @@ template <int DREG>
 int launch_delta_recurrence(const float* prep, long ldp, DeltaDims m, float* state, const int32_t* seq_q_start,
                             const int32_t* seq_slot, float* o_raw, long ldo, int n_seqs, int write_state,
                             cudaStream_t stream) {
-  const int cols = (m.Dv + 31) / 32 * 32;
-  const size_t smem = ((size_t)(m.channel ? 6 : 4) * m.D + (DREG > 0 ? 0 : (size_t)m.D * cols)) * sizeof(float);
+  int cols = (m.Dv + 31) / 32 * 32;
+  auto bytes = [&](int c) { return ((size_t)(m.channel ? 6 : 4) * m.D + (DREG > 0 ? 0 : (size_t)m.D * c)) * sizeof(float); };
+  while (bytes(cols) > 200 * 1024 && cols > 32) cols = (cols / 2 + 31) / 32 * 32;
+  const size_t smem = bytes(cols);
+  if (smem > 200 * 1024) return LLMI_ERR_BAD_SIZE;
   static PerDevice<size_t> allowed;
   if (smem > 48 * 1024 && allowed.here() < smem) {
     if (cudaFuncSetAttribute(delta_recurrence_kernel<DREG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return LLMI_ERR_BAD_SIZE;
     allowed.here() = smem;
   }
-  return launch_pdl(PDL_ATTENTION, delta_recurrence_kernel<DREG>, dim3(m.H, n_seqs), dim3(cols), smem, stream, prep, ldp, m, state,
+  return launch_pdl(PDL_ATTENTION, delta_recurrence_kernel<DREG>, dim3(m.H, n_seqs, (m.Dv + cols - 1) / cols), dim3(cols), smem, stream, prep, ldp, m, state,
                     seq_q_start, seq_slot, o_raw, ldo, write_state);
 }
 
@@ -531,7 +534,6 @@ LLMI_EXPORT int llmi_delta_recurrence(const float* prep, long ldp, int H, int Hk
     if (D == 128) LLMI_QUAD(128);
 #undef LLMI_QUAD
   }
-  if ((size_t)D * ((Dv + 31) / 32 * 32) * 4 + 24 * (size_t)D > 200 * 1024) return LLMI_ERR_BAD_SIZE;
   return launch_delta_recurrence<0>(prep, ldp, m, state, seq_q_start, seq_slot, o_raw, ldo, n_seqs, write_state, stream);
 }
 
