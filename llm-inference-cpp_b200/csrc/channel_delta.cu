@@ -121,6 +121,10 @@ channel_token_prepare_kernel(const ChannelTokenArgs a, const T* __restrict__ w_a
   const int t0 = group * TG;
   float* low = ct_smem;                                  // [R][TG]
   float* part = ct_smem + (size_t)R * TG;                // [warps][64][TG + 1]
+  const int span = (R + CT_WARPS - 1) / CT_WARPS, r_lo = warp * span, r_hi = min(R, r_lo + span);
+  float2 wv[8];                                          // weights wait for nobody: the first eight rows are asked for now
+#pragma unroll
+  for (int j = 0; j < 8; ++j) wv[j] = r_lo + j < r_hi ? ct_pair(w + (size_t)(r_lo + j) * ldw + n0 + 2 * lane) : make_float2(0.f, 0.f);
   pdl_wait();
   for (int i = threadIdx.x; i < R * TG; i += CT_THREADS) {
     const int tt = i / R, r = i - tt * R;                // neighbouring threads read neighbouring columns
@@ -130,29 +134,23 @@ channel_token_prepare_kernel(const ChannelTokenArgs a, const T* __restrict__ w_a
   float2 acc[TG];
 #pragma unroll
   for (int t = 0; t < TG; ++t) acc[t] = make_float2(0.f, 0.f);
-  const int span = (R + CT_WARPS - 1) / CT_WARPS, r_lo = warp * span, r_hi = min(R, r_lo + span);
-  int r = r_lo;
-  for (; r + 8 <= r_hi; r += 8) {
-    float2 wv[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) wv[j] = ct_pair(w + (size_t)(r + j) * ldw + n0 + 2 * lane);
+  for (int r = r_lo; r < r_hi; r += 8) {
+    float2 nxt[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j)
+      nxt[j] = r + 8 + j < r_hi ? ct_pair(w + (size_t)(r + 8 + j) * ldw + n0 + 2 * lane) : make_float2(0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (r + j >= r_hi) break;
 #pragma unroll
       for (int t = 0; t < TG; ++t) {
         const float l = low[(r + j) * TG + t];
         acc[t].x = fmaf(wv[j].x, l, acc[t].x);
         acc[t].y = fmaf(wv[j].y, l, acc[t].y);
       }
-  }
-  for (; r < r_hi; ++r) {
-    const float2 wv = ct_pair(w + (size_t)r * ldw + n0 + 2 * lane);
-#pragma unroll
-    for (int t = 0; t < TG; ++t) {
-      const float l = low[r * TG + t];
-      acc[t].x = fmaf(wv.x, l, acc[t].x);
-      acc[t].y = fmaf(wv.y, l, acc[t].y);
     }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) wv[j] = nxt[j];
   }
   float* mine = part + (size_t)warp * CT_TILE * (TG + 1);
 #pragma unroll

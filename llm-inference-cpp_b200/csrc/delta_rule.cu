@@ -111,6 +111,104 @@ delta_prepare_kernel(const float* __restrict__ proj, long ld, DeltaDims m, const
   }
 }
 
+// The same for many tokens: a warp takes 128 neighbouring channels — a head of q or k, or a piece of v — of DELTA_TILE
+// consecutive tokens, four channels a lane, and keeps the convolution's inputs in registers from token to token; behind them
+// the pieces of decays (channel only), likewise, and the last piece of all makes what a head has one number of.  For heads of
+// up to 128 entries, all parts in whole 16-byte pieces, K taps.
+constexpr int DELTA_TILE = 16, DELTA_TILE_WARPS = 4;
+
+template <int K>
+__global__ void __launch_bounds__(DELTA_TILE_WARPS * 32)
+delta_prepare_tile_kernel(const float* __restrict__ proj, long ld, DeltaDims m, const float* __restrict__ conv_w,
+                          const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ state,
+                          const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos,
+                          const int32_t* __restrict__ seq_q_start, const int32_t* __restrict__ seq_slot,
+                          float* __restrict__ prep, long ldp, const float* __restrict__ z, long ldz, int n_tokens, int pieces) {
+  pdl_launch_dependents();
+  const int piece = blockIdx.y * DELTA_TILE_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * DELTA_TILE, t1 = min(n_tokens, t0 + DELTA_TILE);
+  pdl_wait();
+  if (piece >= pieces) return;
+  const int Nc = m.n_conv(), Nqk = m.n_qk(), n_v = m.H * m.Dv, v_pieces = (n_v + 127) / 128;
+  const int n_g = m.channel ? m.H * m.D : 0, g_pieces = (n_g + 127) / 128;
+  if (piece == pieces - 1) {                             // one number per (token, head)
+    for (int t = t0; t < t1; ++t) {
+      if (tok_seq[t] < 0) continue;
+      const float* row = proj + (size_t)t * ld;
+      float* out = prep + (size_t)t * ldp;
+      for (int h = lane; h < m.H; h += 32) {
+        out[m.beta_at() + h] = 1.0f / (1.0f + expf(-row[Nc + h]));
+        if (!m.channel) out[m.decay_at() + h] = expf(-expf(a_log[h]) * softplus_f(row[Nc + m.H + h] + dt_bias[h]));
+      }
+    }
+    return;
+  }
+  if (piece >= 2 * m.Hk + v_pieces) {                    // decays
+    const int c = (piece - 2 * m.Hk - v_pieces) * 128 + 4 * lane;
+    if (c >= n_g) return;
+    const float a = -expf(a_log[c / m.D]);               // (a head's entries are whole fours)
+    const float4 b = *reinterpret_cast<const float4*>(dt_bias + c);
+    for (int t = t0; t < t1; ++t) {
+      if (tok_seq[t] < 0) continue;
+      const float4 v = *reinterpret_cast<const float4*>(z + (size_t)t * ldz + c);
+      *reinterpret_cast<float4*>(prep + (size_t)t * ldp + m.decay_at() + c) =
+          make_float4(expf(a * softplus_f(v.x + b.x)), expf(a * softplus_f(v.y + b.y)), expf(a * softplus_f(v.z + b.z)),
+                      expf(a * softplus_f(v.w + b.w)));
+    }
+    return;
+  }
+  const bool unit = piece < 2 * m.Hk;
+  const int ch = unit ? piece * m.D + 4 * lane : Nqk + (piece - 2 * m.Hk) * 128 + 4 * lane;
+  const bool mine = unit ? 4 * lane < m.D : ch < Nc;
+  float4 w[K], x[K];                                     // tap j multiplies the input K - 1 - j tokens back; x[j] is that input
+#pragma unroll
+  for (int j = 0; j < K; ++j) {
+    const float* p = conv_w + (size_t)ch * K + j;
+    w[j] = mine ? make_float4(p[0], p[K], p[2 * K], p[3 * K]) : make_float4(0.f, 0.f, 0.f, 0.f);
+    x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const float q_scale = piece < m.Hk ? 1.0f / sqrtf((float)m.D) : 1.0f;
+  int at_seq = -1;
+  for (int t = t0; t < t1; ++t) {
+    const int seq = tok_seq[t];
+    const int slot = seq >= 0 ? seq_slot[seq] : -1;
+    if (slot < 0) {                                      // (the whole warp agrees)
+      at_seq = -1;
+      continue;
+    }
+    if (seq != at_seq) {                                 // a sequence begins in this tile, or the tile in a sequence: its last inputs
+      const int pos = tok_pos[t], r0 = seq_q_start[seq], p0 = pos - (t - r0);
+      const float* carry = state + (size_t)slot * m.state_floats() + m.conv_offset();
+#pragma unroll
+      for (int j = 1; j < K; ++j) {                      // x[j] moves to x[j - 1] below
+        const int p = pos - (K - j);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (p >= 0 && mine) v = p >= p0 ? *reinterpret_cast<const float4*>(proj + (size_t)(r0 + p - p0) * ld + ch)
+                                        : *reinterpret_cast<const float4*>(carry + (size_t)(p - (p0 - (K - 1))) * Nc + ch);
+        x[j] = v;
+      }
+      at_seq = seq;
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < K; ++j) x[j] = x[j + 1];
+    if (mine) x[K - 1] = *reinterpret_cast<const float4*>(proj + (size_t)t * ld + ch);
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+      y.x = fmaf(x[j].x, w[j].x, y.x);
+      y.y = fmaf(x[j].y, w[j].y, y.y);
+      y.z = fmaf(x[j].z, w[j].z, y.z);
+      y.w = fmaf(x[j].w, w[j].w, y.w);
+    }
+    y = make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w));
+    if (unit) {
+      const float sc = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) + 1e-6f) * q_scale;
+      y = make_float4(y.x * sc, y.y * sc, y.z * sc, y.w * sc);
+    }
+    if (mine) *reinterpret_cast<float4*>(prep + (size_t)t * ldp + ch) = y;
+  }
+}
+
 // One thread per (sequence, channel): the inputs of the last taps-1 positions after this step, from the step's own
 // rows or, where the step brought fewer, from what the slab held.
 __global__ void __launch_bounds__(128)
@@ -500,6 +598,18 @@ LLMI_EXPORT int llmi_delta_prepare(const float* proj, long ld, int H, int Hk, in
                                    long ldp, int n_tokens, const float* z, long ldz, cudaStream_t stream) {
   const DeltaDims m{H, Hk, D, Dv, taps, z != nullptr};
   if (n_tokens <= 0 || !delta_dims_ok(m)) return LLMI_ERR_BAD_SIZE;
+  if (n_tokens >= 64 && taps <= 4 && D % 4 == 0 && D <= 128 && Dv % 4 == 0 && ld % 4 == 0 && ldp % 4 == 0 && ldz % 4 == 0 &&
+      m.state_floats() % 4 == 0 && (m.channel == 0 || m.decay_at() % 4 == 0) && !((uintptr_t)proj & 15) && !((uintptr_t)prep & 15) &&
+      !((uintptr_t)state & 15) && !((uintptr_t)z & 15) && !((uintptr_t)dt_bias & 15)) {
+    const int pieces = 2 * m.Hk + (m.H * m.Dv + 127) / 128 + (m.channel ? (m.H * m.D + 127) / 128 : 0) + 1;
+    const dim3 grid((n_tokens + DELTA_TILE - 1) / DELTA_TILE, (pieces + DELTA_TILE_WARPS - 1) / DELTA_TILE_WARPS);
+    if (grid.y <= 65535) {
+      auto kernel = taps == 1 ? delta_prepare_tile_kernel<1> : taps == 2 ? delta_prepare_tile_kernel<2>
+                              : taps == 3 ? delta_prepare_tile_kernel<3> : delta_prepare_tile_kernel<4>;
+      return launch_pdl(PDL_SMALL, kernel, grid, dim3(DELTA_TILE_WARPS * 32), 0, stream, proj, ld, m, conv_w, a_log, dt_bias, state, tok_seq,
+                        tok_pos, seq_q_start, seq_slot, prep, ldp, z, ldz, n_tokens, pieces);
+    }
+  }
   const int pieces = 2 * m.Hk + (m.H * m.Dv + DELTA_V_PIECE - 1) / DELTA_V_PIECE +
                      (m.channel ? (m.H * m.D + DELTA_V_PIECE - 1) / DELTA_V_PIECE : 0);
   if (pieces > 65535) return LLMI_ERR_BAD_SIZE;

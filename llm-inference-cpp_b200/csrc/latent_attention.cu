@@ -45,42 +45,79 @@ __device__ __forceinline__ void rotate_part(const float* __restrict__ src, T* __
   for (int i = rot_dims + me; i < R; i += n) dst[i] = from_f32<T>(src[i]);
 }
 
-// One block per token.  down: fp32 [T, ld]: columns [0, Q) query latent, [Q, Q+C) key/value latent, [Q+C, Q+C+R)
-// the shared key part.  cq (type T) [T, Q] receives the normed query latent; the cache row of (sequence, position)
-// receives [normed c | rotated r].
+// n entries of src, divided by their root mean square and weighted, into dst; the whole block takes part.  A row of up to
+// LN_KEEP entries per thread is read once (and its weights before the wait on the kernel ahead: `w` waits for nobody).
+constexpr int LP_THREADS = 256, LN_KEEP = 6;
 template <typename T>
-__global__ void __launch_bounds__(128)
+__device__ __forceinline__ void normed_part(const float* __restrict__ src, const float* __restrict__ w, int n, float eps, T* __restrict__ dst,
+                                            const float (&wv)[LN_KEEP], float* scratch) {
+  const bool kept = n <= LN_KEEP * LP_THREADS;
+  float v[LN_KEEP], ss = 0.f;
+  if (kept) {
+#pragma unroll
+    for (int j = 0; j < LN_KEEP; ++j) {
+      const int i = threadIdx.x + j * LP_THREADS;
+      v[j] = i < n ? src[i] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < LN_KEEP; ++j) ss = fmaf(v[j], v[j], ss);
+  } else {
+    for (int i = threadIdx.x; i < n; i += LP_THREADS) ss = fmaf(src[i], src[i], ss);
+  }
+  const float sc = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  if (kept) {
+#pragma unroll
+    for (int j = 0; j < LN_KEEP; ++j) {
+      const int i = threadIdx.x + j * LP_THREADS;
+      if (i < n) dst[i] = from_f32<T>(wv[j] * (v[j] * sc));
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += LP_THREADS) dst[i] = from_f32<T>(w[i] * (src[i] * sc));
+  }
+}
+
+// Two blocks per token: the query latent (blockIdx.y 0), and the cache row (1; only where rows are written).  down: fp32 [T,
+// ld]: columns [0, Q) query latent, [Q, Q+C) key/value latent, [Q+C, Q+C+R) the shared key part.  cq (type T) [T, Q]
+// receives the normed query latent; the cache row of (sequence, position) receives [normed c | rotated r].
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS)
 latent_prepare_kernel(const float* __restrict__ down, long ld, int Q, int C, int R, const float* __restrict__ wq,
                       const float* __restrict__ wc, float eps, const float* __restrict__ inv_freq, int rot_dims,
                       const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos, PagedKV kv,
                       T* __restrict__ cache, T* __restrict__ cq, int write_kv, int pairing, float amplitude) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
-  pdl_wait();
-  const int t = blockIdx.x;
-  const int seq = tok_seq[t];
-  T* cq_row = cq + (size_t)t * Q;
-  if (seq < 0) {
-    for (int i = threadIdx.x; i < Q; i += blockDim.x) cq_row[i] = from_f32<T>(0.f);
-    return;
+  const int t = blockIdx.x, seq = tok_seq[t];            // (the step's index block: there before any of its kernels)
+  const bool is_row = blockIdx.y == 1;
+  const int n = is_row ? C : Q;
+  const float* w = is_row ? wc : wq;
+  float wv[LN_KEEP];
+#pragma unroll
+  for (int j = 0; j < LN_KEEP; ++j) {
+    const int i = threadIdx.x + j * LP_THREADS;
+    wv[j] = i < n ? w[i] : 0.f;
   }
   const float* row = down + (size_t)t * ld;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < Q; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-  ss = block_sum(ss, scratch);
-  const float sq = 1.0f / sqrtf(ss / (float)Q + eps);
-  for (int i = threadIdx.x; i < Q; i += blockDim.x) cq_row[i] = from_f32<T>(wq[i] * (row[i] * sq));
-  if (!write_kv) return;
-  const float* c = row + Q;
-  ss = 0.f;
-  for (int i = threadIdx.x; i < C; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
-  ss = block_sum(ss, scratch);
-  const float sc = 1.0f / sqrtf(ss / (float)C + eps);
+  if (!is_row) {
+    T* cq_row = cq + (size_t)t * Q;
+    pdl_wait();
+    if (seq < 0) {
+      for (int i = threadIdx.x; i < Q; i += blockDim.x) cq_row[i] = from_f32<T>(0.f);
+      return;
+    }
+    normed_part<T>(row, wq, Q, eps, cq_row, wv, scratch);
+    return;
+  }
+  if (seq < 0) {
+    pdl_wait();
+    return;
+  }
   const int pos = tok_pos[t];
+  const float* c = row + Q;
   T* dst = cache + kv_row_offset(kv, seq, pos, 0);
-  for (int i = threadIdx.x; i < C; i += blockDim.x) dst[i] = from_f32<T>(wc[i] * (c[i] * sc));
-  const float* r = c + C;
-  rotate_part<T>(r, dst + C, R, inv_freq, rot_dims, pairing, amplitude, pos, threadIdx.x, blockDim.x);
+  pdl_wait();
+  normed_part<T>(c, wc, C, eps, dst, wv, scratch);
+  rotate_part<T>(c + C, dst + C, R, inv_freq, rot_dims, pairing, amplitude, pos, threadIdx.x, blockDim.x);
 }
 
 // The same for a layer whose queries come straight from its input.  proj: fp32 [T, ld]: [ q: H * (D + R) | c: C | r: R ].
@@ -297,10 +334,10 @@ LLMI_EXPORT int llmi_latent_prepare(int dtype, const float* down, long ld, int Q
   if (n_tokens <= 0 || Q <= 0 || C <= 0 || R < 0 || rot_dims < 0 || rot_dims > R || (rot_dims & 1)) return LLMI_ERR_BAD_SIZE;
   PagedKV kv{seq_pages, pages_stride, page_size, 1, C + R};
   if (dtype == LLMI_DTYPE_F32)
-    return launch_pdl(PDL_ROPE, latent_prepare_kernel<float>, n_tokens, 128, 0, stream, down, ld, Q, C, R, wq, wc, eps, inv_freq,
+    return launch_pdl(PDL_ROPE, latent_prepare_kernel<float>, dim3(n_tokens, write_kv ? 2 : 1), dim3(LP_THREADS), 0, stream, down, ld, Q, C, R, wq, wc, eps, inv_freq,
                       rot_dims, tok_seq, tok_pos, kv, (float*)cache, (float*)cq, write_kv, pairing, amplitude);
   if (dtype == LLMI_DTYPE_BF16)
-    return launch_pdl(PDL_ROPE, latent_prepare_kernel<__nv_bfloat16>, n_tokens, 128, 0, stream, down, ld, Q, C, R, wq, wc, eps,
+    return launch_pdl(PDL_ROPE, latent_prepare_kernel<__nv_bfloat16>, dim3(n_tokens, write_kv ? 2 : 1), dim3(LP_THREADS), 0, stream, down, ld, Q, C, R, wq, wc, eps,
                       inv_freq, rot_dims, tok_seq, tok_pos, kv, (__nv_bfloat16*)cache, (__nv_bfloat16*)cq, write_kv, pairing, amplitude);
   return LLMI_ERR_BAD_DTYPE;
 }
